@@ -4,7 +4,7 @@ slots for fixed-size per-request state.  Pure bookkeeping, no tensors.
 Layers whose mixers need the same kind of cache form a group with a page pool of its own:
 full attention keeps every page of a live request; a window group gives a page back as soon
 as every position in it lies more than ``window`` behind the request's stored length, and
-hands it out again.  Block tables are indexed by logical page (position // page_size);
+hands it out again (pages of the ``keep_first`` first positions, which stay visible, are kept).  Block tables are indexed by logical page (position // page_size);
 a page given back leaves -1 behind, which the kernels never index.
 
 Reference: puneethgv/DiSpec dispec/kv/block_manager.py (one group, tables at :22-31, allocate
@@ -43,6 +43,7 @@ class CacheGroupSpec:
     tensors: tuple  # of CacheTensor
     window: int = 0  # 0: all tokens stay
     num_slots: int = 1  # layer caches in the group
+    keep_first: int = 0  # with a window: so many first positions stay as well
 
     @classmethod
     def key_value(cls, num_kv_heads: int, head_dim: int, window: int = 0, num_slots: int = 1):
@@ -58,7 +59,7 @@ class _Request:
     state_slot: int
     num_tokens: int = 0  # tokens whose keys/values are stored
     tables: list[list[int]] = field(default_factory=list)  # per group, logical page -> page id | -1
-    first_live: list[int] = field(default_factory=list)  # per group, first logical page still held
+    first_live: list[int] = field(default_factory=list)  # per group, first logical page not yet given back (behind kept ones)
     reserved: list[int] = field(default_factory=list)  # per group, pages still promised
     renew: list[bool] = field(default_factory=list)  # per group: a released page renews the promise
 
@@ -122,9 +123,10 @@ class CacheManager:
         """Most pages a request ever holds at once in a window group: a step of ``max_chunk``
         tokens needs the window - 1 positions before it and its own, which touch at most one page
         more than they fill; never more than the pages of the ``max_total_len`` positions the
-        request ever stores."""
+        request ever stores.  Pages of kept first positions come on top."""
         w = self.groups[group].window
         bound = (w - 1 + max(1, max_chunk) + self.page_size - 1) // self.page_size + 1
+        bound += self.pages_for(self.groups[group].keep_first)
         return min(bound, self.pages_for(max_total_len))
 
     def largest_chunk(self) -> int:
@@ -133,7 +135,8 @@ class CacheManager:
         cap = 1 << 62
         for spec, pool in zip(self.groups, self.pools):
             if spec.window > 0:
-                cap = min(cap, (pool.num_pages - 1) * self.page_size - spec.window + 1)
+                kept = self.pages_for(spec.keep_first)
+                cap = min(cap, (pool.num_pages - 1 - kept) * self.page_size - spec.window + 1)
         return cap
 
     # ---------------------------------------------------------------------- lifecycle
@@ -218,6 +221,8 @@ class CacheManager:
             first_needed = max(0, num_tokens - spec.window + 1)
             keep_from = first_needed // self.page_size
             table = r.tables[g]
+            kept = self.pages_for(spec.keep_first)
+            r.first_live[g] = max(r.first_live[g], min(kept, len(table)))
             while r.first_live[g] < min(keep_from, len(table)):
                 j = r.first_live[g]
                 page = table[j]

@@ -30,6 +30,11 @@ class ModelConfig:
     def to_dict(self) -> dict:
         raise NotImplementedError
 
+    def with_tensor_shapes(self, source) -> "ModelConfig":
+        """The configuration with the sizes that only the checkpoint's tensors give (``source``: ``names()``
+        and ``shape(name)``); most architectures have none."""
+        return self
+
     def flat(self) -> dict:
         """Scalars only, for logs and benchmark records."""
         out = {}

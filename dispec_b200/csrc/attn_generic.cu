@@ -8,6 +8,7 @@
 // over tiles of 128 keys.  Keys have D dimensions and values Dv (the pools have their own widths).
 // With `mask_mode` 1 the number `window` is a chunk size instead: position p sees the keys of its own
 // chunk, floor(p / size) * size <= b <= p (chunks counted from position 0 of the sequence).
+// With `keep_first` = F the keys b < F are seen as well, however far behind the window they lie.
 // With `sink` the softmax has one more, imaginary key and no value for it: the weights are
 // exp(s_j) / (exp(z) + sum exp(s_j)), z = sink_values[head] (unscaled), or 0 without `sink_values`;
 // the running pair starts at (m, l) = (z, 1) instead of (-inf, 0).
@@ -33,7 +34,7 @@ attn_generic_kernel(const T* __restrict__ q, long q_stride, const T* __restrict_
                     int pt_stride, const int* __restrict__ positions,
                     const int* __restrict__ seq_of_token, void* __restrict__ out, int out_dtype, long out_stride,
                     int H, int KVH, int D, int Dv, int page_size, int num_pages, int window, int mask_mode,
-                    float scale, int sink, const float* __restrict__ sink_values,
+                    int keep_first, float scale, int sink, const float* __restrict__ sink_values,
                     const float* __restrict__ turn_freq, int* err) {
   extern __shared__ float smem[];
   float* qs = smem;                       // [GCHUNK][D]
@@ -48,8 +49,10 @@ attn_generic_kernel(const T* __restrict__ q, long q_stride, const T* __restrict_
   if (pos < 0) return;
   const int seq = seq_of_token[t];
   const int G = H / KVH;
-  const int lo = window > 0 ? (mask_mode == 1 ? (pos / window) * window : max(0, pos - window + 1)) : 0;
-  const int hi = pos;
+  int lo = window > 0 ? (mask_mode == 1 ? (pos / window) * window : max(0, pos - window + 1)) : 0;
+  if (lo <= keep_first) lo = 0;
+  const int front = min(keep_first, lo), nfront = (front + THREADS - 1) / THREADS;  // kept keys, and the tiles they take
+  const int hi = pos, ntiles = nfront + (hi - lo) / THREADS + 1;
   const int* table = page_table + (size_t)seq * pt_stride;
 
   for (int g0 = 0; g0 < G; g0 += GCHUNK) {
@@ -69,9 +72,11 @@ attn_generic_kernel(const T* __restrict__ q, long q_stride, const T* __restrict_
     }
     __syncthreads();
 
-    for (int kt = lo; kt <= hi; kt += THREADS) {
+    for (int tile = 0; tile < ntiles; ++tile) {
+      const int kt = tile < nfront ? tile * THREADS : lo + (tile - nfront) * THREADS;
+      const int last = tile < nfront ? front - 1 : hi;
       const int key = kt + tid;
-      const bool valid = key <= hi;
+      const bool valid = key <= last;
       float s[GCHUNK];
 #pragma unroll
       for (int g = 0; g < GCHUNK; ++g) s[g] = -INFINITY;
@@ -131,7 +136,7 @@ attn_generic_kernel(const T* __restrict__ q, long q_stride, const T* __restrict_
         for (int j = 0; j < DPT; ++j) acc[g][j] *= alpha[g];
       }
       // weighted sum of values: thread owns dims tid, tid+128, ...
-      const int nkeys = min(THREADS, hi - kt + 1);
+      const int nkeys = min(THREADS, last - kt + 1);
       for (int j = 0; j < nkeys; ++j) {
         const long vo = slot[j];
         if (vo < 0) continue;
@@ -184,8 +189,8 @@ extern "C" int dsp_attn_generic(const void* q, long q_stride, const void* k_pool
                                 const void* v_pool, const int* page_table, int pt_stride,
                                 const int* positions, const int* seq_of_token, void* out,
                                 long out_stride, int T, int H, int KVH, int D, int Dv, int page_size,
-                                int num_pages, int window, int mask_mode, float scale, int sink,
-                                const float* sink_values, const float* turn_freq, int dtype, int out_dtype,
+                                int num_pages, int window, int mask_mode, int keep_first, float scale,
+                                int sink, const float* sink_values, const float* turn_freq, int dtype, int out_dtype,
                                 cudaStream_t stream) {
   if (T == 0) return 0;
   DSP_REQUIRE(KVH > 0 && H % KVH == 0, "dsp_attn_generic: H=%d is not a multiple of KVH=%d", H, KVH);
@@ -194,6 +199,7 @@ extern "C" int dsp_attn_generic(const void* q, long q_stride, const void* k_pool
               THREADS * DPT);
   DSP_REQUIRE(KVH <= 65535, "dsp_attn_generic: too many KV heads");
   DSP_REQUIRE(mask_mode == 0 || mask_mode == 1, "dsp_attn_generic: unknown mask mode %d", mask_mode);
+  DSP_REQUIRE(keep_first >= 0, "dsp_attn_generic: keep_first=%d", keep_first);
   DSP_REQUIRE(!turn_freq || Dv % 2 == 0, "dsp_attn_generic: values of an odd width %d cannot be turned", Dv);
   int* err = dsp_device_error_ptr();
   DSP_REQUIRE(err != nullptr, "dsp_attn_generic: no device error word");
@@ -210,7 +216,7 @@ extern "C" int dsp_attn_generic(const void* q, long q_stride, const void* k_pool
     attn_generic_kernel<float><<<grid, THREADS, smem, stream>>>(
         (const float*)q, q_stride, (const float*)k_pool, (const float*)v_pool, page_table, pt_stride,
         positions, seq_of_token, out, out_dtype, out_stride, H, KVH, D, Dv, page_size, num_pages, window,
-        mask_mode, scale, sink, sink_values, turn_freq, err);
+        mask_mode, keep_first, scale, sink, sink_values, turn_freq, err);
   } else if (dtype == DSP_BF16) {
     static size_t configured = 0;
     if (smem > configured) {
@@ -221,7 +227,7 @@ extern "C" int dsp_attn_generic(const void* q, long q_stride, const void* k_pool
     attn_generic_kernel<bf16><<<grid, THREADS, smem, stream>>>(
         (const bf16*)q, q_stride, (const bf16*)k_pool, (const bf16*)v_pool, page_table, pt_stride,
         positions, seq_of_token, out, out_dtype, out_stride, H, KVH, D, Dv, page_size, num_pages, window,
-        mask_mode, scale, sink, sink_values, turn_freq, err);
+        mask_mode, keep_first, scale, sink, sink_values, turn_freq, err);
   } else {
     DSP_REQUIRE(false, "dsp_attn_generic: unknown dtype %d", dtype);
   }

@@ -1,6 +1,6 @@
 // Tensor-core attention (mma.sync m16n8k16, bfloat16 operands, 32-bit scores, softmax and sums)
 // over paged keys of width DSP_DK and values of width DSP_DV, with a sliding window or a chunked
-// mask and an optional sink in the softmax (one more key with no value, of score 0 or, with
+// mask, kept first keys and an optional sink in the softmax (one more key with no value, of score 0 or, with
 // `sink_values`, of the head's own unscaled score z: the running pair of the online softmax starts
 // at (max, sum) = (z, 1) instead of (-inf, 0)).  With `turn_freq` every head's result is turned
 // back, pair (m, m + DV/2) by -p * turn_freq[m] (values that were stored turned by their own
@@ -12,7 +12,8 @@
 // a key row is found through the request's page table, a page id outside the pool is recorded
 // and its keys are hidden from every row.  The query at position p sees keys j with
 // p - window < j <= p (window 0: every j <= p; mask_mode 1: the keys of p's own chunk of `window`
-// positions, floor(p / window) * window <= j <= p); positions follow from the request's stored length
+// positions, floor(p / window) * window <= j <= p) and, with `keep_first` = F, the keys j < F as well, which
+// come in key tiles of their own in front of the others where the window has left them behind; positions follow from the request's stored length
 // (ctx_len) and the number of tokens it brings.  A request of length 0 (a padding row of a
 // captured step) is skipped.
 //
@@ -60,7 +61,7 @@ attn_sink_mma_kernel(const bf16* __restrict__ q, long ldq, const bf16* __restric
                      const bf16* __restrict__ v_pool, const int* __restrict__ page_table, int pt_stride,
                      const int* __restrict__ q_start, const int* __restrict__ ctx_len,
                      const int* __restrict__ tile_seq, const int* __restrict__ tile_tok0, void* __restrict__ out, int out_f32,
-                     long ldo, int H, int G, int tpt, int page_size, int num_pages, int window, int mask_mode,
+                     long ldo, int H, int G, int tpt, int page_size, int num_pages, int window, int mask_mode, int keep_first,
                      float scale_log2, int sink, const float* __restrict__ sink_values,
                      const float* __restrict__ turn_freq, int tile_offset, int splits,
                      float* __restrict__ part_o, float* __restrict__ part_ml, int* err) {
@@ -80,12 +81,17 @@ attn_sink_mma_kernel(const bf16* __restrict__ q, long ldq, const bf16* __restric
   auto first_seen = [&](int p) {
     return window > 0 ? (mask_mode == 1 ? (p / window) * window : max(0, p - window + 1)) : 0;
   };
-  const int lo = first_seen(pos0);
-  const int nkt_all = (p1 - lo) / BN + 1;
+  int lo = first_seen(pos0);
+  if (lo <= keep_first) lo = 0;
+  const int front = min(keep_first, lo), nfront = (front + BN - 1) / BN;  // kept keys behind every window, their tiles
+  const int nkt_all = nfront + (p1 - lo) / BN + 1;
   const int kt0 = (int)((long)nkt_all * split / splits), kt1 = (int)((long)nkt_all * (split + 1) / splits);
   const int nkt = kt1 - kt0;  // this block's key tiles: kt0 .. kt1 - 1 (none: it leaves an empty partial)
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int* table = page_table + (size_t)seq * pt_stride;
+  // first key of tile kt of this block, and the last key that the tile stands for
+  auto tile_first = [&](int kt) { return kt0 + kt < nfront ? (kt0 + kt) * BN : lo + (kt0 + kt - nfront) * BN; };
+  auto tile_last = [&](int kt) { return kt0 + kt < nfront ? front - 1 : p1; };
 
   for (int c = tid; c < BM * (DK / 8); c += 128) {
     const int r = c / (DK / 8), d = (c % (DK / 8)) * 8;
@@ -98,14 +104,14 @@ attn_sink_mma_kernel(const bf16* __restrict__ q, long ldq, const bf16* __restric
   // returns whether one of this thread's key rows had a page id outside the pool
   auto load = [&](int stage, int kt) {
     int bad = 0;
-    const int j0 = lo + (kt0 + kt) * BN;
+    const int j0 = tile_first(kt), jend = tile_last(kt);
     bf16* ks = Ks + stage * BN * LDK;
     bf16* vs = Vs + stage * BN * LDV;
     // two threads a key row: the page is looked up once a row, the row's 16-byte pieces alternate
     const int r = tid >> 1;
     const int j = j0 + r;
     long row = -1;
-    if (j <= p1) {
+    if (j <= jend) {
       const int page = table[j / page_size];
       if (page < 0 || page >= num_pages) {
         atomicOr(err, DSP_ERR_BAD_PAGE);
@@ -174,7 +180,7 @@ attn_sink_mma_kernel(const bf16* __restrict__ q, long ldq, const bf16* __restric
         mma16816(s[j + 1], a, b[2], b[3]);
       }
     }
-    const int j0 = lo + (kt0 + kt) * BN;
+    const int j0 = tile_first(kt), jend = tile_last(kt);
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int i = 0; i < BN / 8; ++i)
@@ -182,7 +188,7 @@ attn_sink_mma_kernel(const bf16* __restrict__ q, long ldq, const bf16* __restric
       for (int e = 0; e < 4; ++e) {
         const int j = j0 + i * 8 + (lane & 3) * 2 + (e & 1);
         const int p = e < 2 ? pa : pb;
-        const bool seen = !hide_all && j <= p && j >= (e < 2 ? la : lb);
+        const bool seen = !hide_all && j <= p && j <= jend && (j >= (e < 2 ? la : lb) || j < keep_first);
         s[i][e] = seen ? s[i][e] * scale_log2 : -INFINITY;
         mx[e >> 1] = fmaxf(mx[e >> 1], s[i][e]);
       }
@@ -280,12 +286,12 @@ attn_sink_mma_kernel(const bf16* __restrict__ q, long ldq, const bf16* __restric
 extern "C" int DSP_CAT(dsp_attn_sink_mma_k, DSP_DK, _v, DSP_DV)(
     const void* q, long ldq, const void* k_pool, const void* v_pool, const int* page_table, int pt_stride,
     const int* q_start, const int* ctx_len, const int* tile_seq, const int* tile_tok0, int tile_offset, int num_tiles,
-    void* out, int out_f32, long ldo, int H, int G, int tpt, int page_size, int num_pages, int window, int mask_mode, float scale,
-    int sink, const float* sink_values, const float* turn_freq, int splits, float* part_o, float* part_ml, int* err,
+    void* out, int out_f32, long ldo, int H, int G, int tpt, int page_size, int num_pages, int window, int mask_mode, int keep_first,
+    float scale, int sink, const float* sink_values, const float* turn_freq, int splits, float* part_o, float* part_ml, int* err,
     cudaStream_t stream) {
   if (num_tiles == 0) return 0;
   if (G <= 0 || H % G || tpt <= 0 || tpt * (H / G) > BM || G > 65535 || page_size <= 0 || !err) return 2;
-  if (mask_mode < 0 || mask_mode > 1) return 2;
+  if (mask_mode < 0 || mask_mode > 1 || keep_first < 0) return 2;
   if (splits < 1 || splits > 32 || (splits > 1 && (!part_o || !part_ml))) return 2;
   if (((uintptr_t)q % 16) || ((uintptr_t)k_pool % 16) || ((uintptr_t)v_pool % 16) || ((uintptr_t)out % (out_f32 ? 8 : 4)) || ldq % 8 || ldo % 2)
     return 3;
@@ -299,7 +305,7 @@ extern "C" int DSP_CAT(dsp_attn_sink_mma_k, DSP_DK, _v, DSP_DV)(
   const cudaError_t e = launch_plain(attn_sink_mma_kernel, dim3(num_tiles, G, splits), dim3(128), smem, stream, (const bf16*)q, ldq,
                                      (const bf16*)k_pool, (const bf16*)v_pool, page_table, pt_stride, q_start, ctx_len,
                                      tile_seq, tile_tok0, out, out_f32, ldo, H, G, tpt, page_size, num_pages, window,
-                                     mask_mode, scale * 1.4426950408889634f, sink, sink_values, turn_freq, tile_offset,
+                                     mask_mode, keep_first, scale * 1.4426950408889634f, sink, sink_values, turn_freq, tile_offset,
                                      splits, part_o, part_ml, err);
   return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : 1;
 }

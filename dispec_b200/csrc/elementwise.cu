@@ -229,15 +229,20 @@ extern "C" int dsp_rmsnorm(void* x, const void* delta, const void* w, void* y, c
   return 0;
 }
 
-// ------------------------------------------------------------------------------- SwiGLU
-// out[t, i] = silu(gate(t, i)) * up(t, i), silu(g) = g / (1 + exp(-g)), in 32-bit.
+// ------------------------------------------------------------------------------- gated units
+// out[t, i] = act(gate(t, i)) * up(t, i) in 32-bit: act 0 is silu(g) = g / (1 + exp(-g)), act 1 the tanh
+// form of gelu, 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))).
 // block == 0: gu row = [all gates | all ups].  block == b > 0: gates and ups interleaved in blocks
 // of b columns: gate(t, i) at column (i / b) * 2b + i % b, up(t, i) b columns further.
 __device__ __forceinline__ size_t gate_column(int i, int inter, int block) {
   return block ? (size_t)(i / block) * 2 * block + i % block : (size_t)i;
 }
+__device__ __forceinline__ float unit_act(float g, int act) {
+  if (act == 1) return 0.5f * g * (1.f + tanhf(0.7978845608028654f * fmaf(0.044715f * g * g, g, g)));
+  return g / (1.f + expf(-g));
+}
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int inter, int block) {
+__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int inter, int block, int act) {
   const size_t t = blockIdx.x;
   const T* row = gu + t * 2 * (size_t)inter;
   const int up_off = block ? block : inter;
@@ -246,14 +251,14 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
     const size_t gc = gate_column(i, inter, block);
     const float gv = to_f32(row[gc]);
     const float uv = to_f32(row[gc + up_off]);
-    o[i] = from_f32<T>(gv / (1.f + expf(-gv)) * uv);
+    o[i] = from_f32<T>(unit_act(gv, act) * uv);
   }
 }
 
 template <typename T>
 __global__ void __launch_bounds__(256)
 swiglu_vec_kernel(const T* __restrict__ gu, T* __restrict__ out, int inter, size_t total_vecs,
-                  int block) {
+                  int block, int act) {
   constexpr int N = Vec16<T>::N;
   pdl_launch_dependents();
   pdl_wait();
@@ -273,15 +278,16 @@ swiglu_vec_kernel(const T* __restrict__ gu, T* __restrict__ out, int inter, size
 #pragma unroll
     for (int k = 0; k < N; ++k) {
       const float gv = to_f32(g[k]);
-      o[k] = from_f32<T>(gv / (1.f + expf(-gv)) * to_f32(u[k]));
+      o[k] = from_f32<T>(unit_act(gv, act) * to_f32(u[k]));
     }
     reinterpret_cast<uint4*>(out + t * (size_t)inter)[c] = oraw;
   }
 }
 
-extern "C" int dsp_swiglu(const void* gate_up, void* out, int T, int inter, int block, int dtype,
+extern "C" int dsp_swiglu(const void* gate_up, void* out, int T, int inter, int block, int act, int dtype,
                           cudaStream_t stream) {
   if (T == 0) return 0;
+  DSP_REQUIRE(act == 0 || act == 1, "dsp_swiglu: unknown activation %d", act);
   DSP_REQUIRE(block >= 0 && (block == 0 || inter % block == 0),
               "dsp_swiglu: interleave block %d does not divide %d", block, inter);
   DSP_REQUIRE(dtype == DSP_F32 || dtype == DSP_BF16, "dsp_swiglu: unknown dtype %d", dtype);
@@ -292,18 +298,18 @@ extern "C" int dsp_swiglu(const void* gate_up, void* out, int T, int inter, int 
     const size_t cap = (size_t)(dsp_num_sms() > 0 ? dsp_num_sms() : 1) * 16;  // grid-stride loop beyond that
     const int blocks = (int)((total + 255) / 256 > cap ? cap : (total + 255) / 256);
     if (dtype == DSP_F32)
-      launch_pdl(swiglu_vec_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gate_up, (float*)out, inter, total, block);
+      launch_pdl(swiglu_vec_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gate_up, (float*)out, inter, total, block, act);
     else
-      launch_pdl(swiglu_vec_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16*)gate_up, (bf16*)out, inter, total, block);
+      launch_pdl(swiglu_vec_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16*)gate_up, (bf16*)out, inter, total, block, act);
     DSP_CHECK_LAUNCH("dsp_swiglu");
     return 0;
   }
   const int chunks = (inter + 255) / 256;
   dim3 grid(T, chunks > 64 ? 64 : chunks);
   if (dtype == DSP_F32)
-    swiglu_kernel<float><<<grid, 256, 0, stream>>>((const float*)gate_up, (float*)out, inter, block);
+    swiglu_kernel<float><<<grid, 256, 0, stream>>>((const float*)gate_up, (float*)out, inter, block, act);
   else
-    swiglu_kernel<bf16><<<grid, 256, 0, stream>>>((const bf16*)gate_up, (bf16*)out, inter, block);
+    swiglu_kernel<bf16><<<grid, 256, 0, stream>>>((const bf16*)gate_up, (bf16*)out, inter, block, act);
   DSP_CHECK_LAUNCH("dsp_swiglu");
   return 0;
 }

@@ -37,7 +37,7 @@ constexpr int W_BYTES = ROWS_W * BK * 2;
 // warp 0: TMA; then ISSUERS warps whose first lanes issue the products (the first of them also owns
 // the tensor memory); then four epilogue warps
 constexpr int MAX_SPLITS = 8;
-enum { EPI_PLAIN = 0, EPI_SWIGLU = 1 };
+enum { EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_GEGLU = 2 };
 
 template <int NB> struct Cfg {
   static constexpr int X_BYTES = NB * BK * 2;
@@ -133,6 +133,14 @@ __device__ __forceinline__ void finish(const Args& a, float v, int m, int n) {
 // 64 rows of A made the epilogue of the gate/up product 3.9 us long.
 __device__ __forceinline__ float silu_times(float gate, float up) {
   return __fdividef(gate, 1.f + __expf(-gate)) * up;
+}
+// the tanh form of gelu(gate), times up: 0.5 (1 + tanh(y)) = 1 / (1 + exp(-2 y))
+__device__ __forceinline__ float gelu_times(float gate, float up) {
+  const float y = 0.7978845608028654f * fmaf(0.044715f * gate * gate, gate, gate);
+  return __fdividef(gate, 1.f + __expf(-2.f * y)) * up;
+}
+__device__ __forceinline__ float unit_times(float gate, float up, bool gelu) {
+  return gelu ? gelu_times(gate, up) : silu_times(gate, up);
 }
 
 // four consecutive values of a row, as 32-bit floats
@@ -344,7 +352,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
   // the block (a warp reaches the 32 lanes of tensor memory that its index modulo 4 names).
   const int quarter = warp & 3;
   const int row = quarter * 32 + lane;
-  const bool swiglu = a.epilogue == EPI_SWIGLU;
+  const bool swiglu = a.epilogue != EPI_PLAIN, gelu = a.epilogue == EPI_GEGLU;
   // The scales of a norm whose gain is already in A: rsqrt(mean square + eps) of the rows of
   // norm_src, by the four epilogue warps (rows in turn, 16-byte loads, 32-bit sums) while the
   // products run.  Called after the wait on the predecessor, which wrote those rows.
@@ -520,7 +528,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
             const float gate = low ? x0 : other, up = low ? other : x1;
             const int m = h0 + (low ? m0 : m0 + 1);
             if (m < a.M && n_ok)
-              reinterpret_cast<TOut*>(a.C)[(size_t)m * a.ldc + col] = from_f32<TOut>(silu_times(gate, up));
+              reinterpret_cast<TOut*>(a.C)[(size_t)m * a.ldc + col] = from_f32<TOut>(unit_times(gate, up, gelu));
           }
         } else {
 #pragma unroll
@@ -639,8 +647,8 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
             if ((lane & 4) == 0 && n4 + 16 < a.N) {
               const int col = ((blockIdx.x * ROWS_W + (lane >> 3) * 32) >> 1) + 4 * (lane & 3);
               store4(reinterpret_cast<TOut*>(a.C) + (size_t)m * a.ldc + col,
-                     make_float4(silu_times(total.x, up.x), silu_times(total.y, up.y), silu_times(total.z, up.z),
-                                 silu_times(total.w, up.w)));
+                     make_float4(unit_times(total.x, up.x, gelu), unit_times(total.y, up.y, gelu),
+                                 unit_times(total.z, up.z, gelu), unit_times(total.w, up.w, gelu)));
             }
           } else if (n_ok) {
             float4 res = res4[0];
@@ -748,7 +756,7 @@ extern "C" int dsp_gemm_stream_stamps_read(unsigned long long* out, long n) {
 }
 #endif
 
-// epilogue: 0 plain (bias, residual allowed); 1 SwiGLU over W rows alternating in blocks of 16
+// epilogue: 0 plain (bias, residual allowed); 1 SwiGLU (2: gelu in its tanh form instead of silu) over W rows alternating in blocks of 16
 // (C is [M, N/2]; no bias, no residual).  target_ctas: resident CTA slots the launch may fill by
 // splitting K (0: one per SM).  late_trigger_bytes: a product that streams at least this many bytes
 // of W lets the next kernel start only when its own last tile is on its way (what the next kernels
@@ -774,6 +782,7 @@ extern "C" int dsp_gemm_stream(const void* A, long lda, const void* W, const voi
   DSP_REQUIRE(K > 0 && K % 8 == 0 && lda % 8 == 0, "dsp_gemm_stream: K=%d and the row stride must be multiples of 8", K);
   DSP_REQUIRE(((uintptr_t)A % 16) == 0 && ((uintptr_t)W % 16) == 0, "dsp_gemm_stream: operands must be 16-byte aligned");
   DSP_REQUIRE(out_dtype == DSP_BF16 || out_dtype == DSP_F32, "dsp_gemm_stream: unknown output dtype %d", out_dtype);
+  DSP_REQUIRE(epilogue >= EPI_PLAIN && epilogue <= EPI_GEGLU, "dsp_gemm_stream: unknown epilogue %d", epilogue);
   DSP_REQUIRE(epilogue == EPI_PLAIN || (N % 32 == 0 && bias == nullptr && residual == nullptr),
               "dsp_gemm_stream: the SwiGLU epilogue needs N in whole blocks of 32 and no bias or residual");
   int* err = dsp_device_error_ptr();

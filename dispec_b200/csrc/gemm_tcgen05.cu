@@ -27,7 +27,7 @@ constexpr int TMEM_COLS = 512;  // two accumulators of 256 columns
 constexpr int EPI_WARPS = 4;
 constexpr int THREADS = 32 * (2 + EPI_WARPS);
 
-enum { EPI_PLAIN = 0, EPI_SWIGLU = 1 };
+enum { EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_GEGLU = 2 };
 
 struct Epilogue {
   int epilogue;
@@ -46,11 +46,20 @@ struct Epilogue {
 __device__ __forceinline__ float silu_times(float gate, float up) {
   return __fdividef(gate, 1.f + __expf(-gate)) * up;
 }
+// the tanh form of gelu(gate), times up: 0.5 (1 + tanh(y)) = 1 / (1 + exp(-2 y))
+__device__ __forceinline__ float gelu_times(float gate, float up) {
+  const float y = 0.7978845608028654f * fmaf(0.044715f * gate * gate, gate, gate);
+  return __fdividef(gate, 1.f + __expf(-2.f * y)) * up;
+}
+__device__ __forceinline__ float unit_times(float gate, float up, bool gelu) {
+  return gelu ? gelu_times(gate, up) : silu_times(gate, up);
+}
 
 template <typename TOut>
 __device__ __forceinline__ void store_row_chunk(const Epilogue& e, const uint32_t (&v)[32], int row, int col) {
   if (row >= e.M || col >= e.N) return;
-  if (e.epilogue == EPI_SWIGLU) {
+  if (e.epilogue != EPI_PLAIN) {
+    const bool gelu = e.epilogue == EPI_GEGLU;
     // W rows alternate in blocks of 16: this chunk holds 16 gates and the 16 ups of the same outputs
     if (col + 32 > e.N) return;
     TOut* dst = reinterpret_cast<TOut*>(e.C) + (size_t)row * e.ldc + (col >> 1);
@@ -62,7 +71,7 @@ __device__ __forceinline__ void store_row_chunk(const Epilogue& e, const uint32_
 #pragma unroll
         for (int t = 0; t < 8; ++t) {
           const float g = __uint_as_float(v[j * 8 + t]), u = __uint_as_float(v[16 + j * 8 + t]);
-          ob[t] = __float2bfloat16(silu_times(g, u));
+          ob[t] = __float2bfloat16(unit_times(g, u, gelu));
         }
         reinterpret_cast<uint4*>(dst)[j] = oraw;
       }
@@ -70,7 +79,7 @@ __device__ __forceinline__ void store_row_chunk(const Epilogue& e, const uint32_
 #pragma unroll  // constant indices: the accumulators stay in registers
       for (int t = 0; t < 16; ++t) {
         const float g = __uint_as_float(v[t]), u = __uint_as_float(v[16 + t]);
-        dst[t] = from_f32<TOut>(silu_times(g, u));
+        dst[t] = from_f32<TOut>(unit_times(g, u, gelu));
       }
     }
     return;
@@ -578,7 +587,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
 }  // namespace
 
 // bfloat16 A [M, K] (row stride lda) and W [N, K] (contiguous); C and residual bfloat16 or float32.
-// epilogue 1: SwiGLU over W rows alternating in blocks of 16 (16 gate rows, their 16 up rows):
+// epilogue 1: SwiGLU (2: gelu in its tanh form instead of silu) over W rows alternating in blocks of 16 (16 gate rows, their 16 up rows):
 // C is [M, N/2], no bias, no residual.
 extern "C" int dsp_gemm_tcgen05(const void* A, long lda, const void* W, const void* bias, const void* residual,
                                 long ldr, void* C, long ldc, int M, int N, int K, int out_dtype, int pair_mode,
@@ -590,6 +599,7 @@ extern "C" int dsp_gemm_tcgen05(const void* A, long lda, const void* W, const vo
   int* err = dsp_device_error_ptr();
   DSP_REQUIRE(err != nullptr, "dsp_gemm_tcgen05: no device error word");
   CUtensorMap map_a, map_w;  // encoded below, once the tile shape is known (an encoding costs the host a microsecond)
+  DSP_REQUIRE(epilogue >= EPI_PLAIN && epilogue <= EPI_GEGLU, "dsp_gemm_tcgen05: unknown epilogue %d", epilogue);
   DSP_REQUIRE(epilogue == EPI_PLAIN || (N % 32 == 0 && bias == nullptr && residual == nullptr),
               "dsp_gemm_tcgen05: the SwiGLU epilogue needs N in whole blocks of 32 and no bias or residual");
   Epilogue e;

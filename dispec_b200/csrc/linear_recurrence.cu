@@ -5,7 +5,7 @@
 //
 // The state of a request lives in its state slot between steps, so a prompt can be cut into
 // portions anywhere and decoded tokens continue from what the prompt left.  What a_t, b_t and
-// q_t are is the mixer's business; two forms are built in, both computed here from the raw
+// q_t are is the mixer's business; four forms are built in, all computed here from the raw
 // rows of the mixer's fused projection (float or bfloat16), in 32-bit:
 //
 //   FIXED_DECAY   a_t = decay[head] (one number per head); q_t and b_t are the projected query
@@ -14,21 +14,28 @@
 //                 with `act` = 1 the raw query, key and value pass through silu first
 //   FORGET_GATE   a_t = f_t = lower + (1 - lower) * sigmoid(raw_f + bias), b_t = 1 - f_t,
 //                 q_t = silu(raw_q)      (lower and bias per head and channel)
+//   KEY_DECAY     q_t = raw_q * q_scale, b_t = raw_k * key_scale, a_t = sigmoid(z)^power with z = M r + bias
+//                 per head and channel, r the `rank` columns of the row from `low_off` on and M given
+//                 transposed ([rank, H * dim])
+//   STEP_DECAY    rows of floats; q_t and b_t are columns shared by the heads of a group, a_t one number per
+//                 token and head and the value scaled by another (`steps`); o_t gets skip[head] * v_t on top:
+//                     S_t = a S_(t-1) + step b_t v_t^T,   o_t = S_t^T q_t + skip v_t
 //
 // One block per (request, head, tile of value columns).  A thread holds ROWS state rows of one
-// column in registers; the SLICES threads that share a column sit in adjacent lanes and add
-// their partial outputs by shuffles.  Tokens are staged through shared memory in rounds of
-// `tokens_per_round`.  The recurrence is sequential in the tokens of a request, so what can be
-// done ahead of it is: for portions of prompts a first, fully parallel kernel writes q_t, b_t
-// (and a_t) of every token as floats, and the recurrence kernel only streams them in with
+// column in registers, four neighbouring rows at a time; the SLICES threads that share a column sit
+// in adjacent lanes and add their partial outputs by shuffles.  Tokens are staged through shared
+// memory in rounds of `tokens_per_round`.  The recurrence is sequential in the tokens of a request,
+// so what can be done ahead of it is: for portions of prompts a first, fully parallel kernel writes
+// q_t, b_t (and a_t) of every token as floats, and the recurrence kernel only streams them in with
 // cp.async, the next round arriving while the current one is computed; single tokens are
-// transformed as they are staged, in one kernel.  A request whose first row carries a negative
+// transformed as they are staged, in one kernel (STEP_DECAY streams the rows themselves always).  A request whose first row carries a negative
 // position (a padding row of a captured step) is skipped: its state slot belongs to someone else.
 #include "common.cuh"
 
 namespace {
 
-enum { FIXED_DECAY = 0, FORGET_GATE = 1 };
+enum { FIXED_DECAY = 0, FORGET_GATE = 1, KEY_DECAY = 2, STEP_DECAY = 3 };
+enum { SCALAR_DECAY = 0, VECTOR_DECAY = 1, TOKEN_DECAY = 2 };  // what a_t is: kinds of the kernel
 constexpr int THREADS = 256;
 
 struct RecurrenceArgs {
@@ -43,8 +50,14 @@ struct RecurrenceArgs {
   int rot;
   float key_scale;
   int act;  // 1: silu on the raw query, key and value (FIXED_DECAY)
-  const float* gate_bias;  // [H * dim]           FORGET_GATE
+  const float* gate_bias;  // [H * dim]           FORGET_GATE, KEY_DECAY
   const float* lower;      // [H * dim]           FORGET_GATE
+  const float* gate_map;   // [rank, H * dim]     KEY_DECAY
+  int low_off, rank;       //                     KEY_DECAY
+  float q_scale, power;    //                     KEY_DECAY
+  const float* steps;      // [T, 2, H]           STEP_DECAY: factor on the value, decay
+  const float* skip;       // [H]                 STEP_DECAY
+  int heads_per_group;     //                     STEP_DECAY (1 otherwise)
   float* state;            // [slots, H, dim, vdim]
   const int* state_slot;   // [S]
   const int* q_start;      // [S + 1]
@@ -56,6 +69,11 @@ struct RecurrenceArgs {
   int cols_per_block;    // threads / slices
   int tokens_per_round;
 };
+
+// sigmoid(z)^power by way of ln sigmoid(z) = -(ln(1 + e^-|z|) + max(-z, 0))
+__device__ __forceinline__ float sigmoid_power(float z, float power) {
+  return expf(-power * (log1pf(expf(-fabsf(z))) + fmaxf(-z, 0.f)));
+}
 
 // q_t, b_t and a_t of element (token, head, i) from the raw projection row, in 32-bit.
 __device__ __forceinline__ void transform(const RecurrenceArgs& p, int token, int head, int i, float& qv,
@@ -87,6 +105,13 @@ __device__ __forceinline__ void transform(const RecurrenceArgs& p, int token, in
       bv = i < half ? bv * cs - k2 * sn : bv * cs + k2 * sn;
     }
     bv *= p.key_scale;
+  } else if (p.mode == KEY_DECAY) {
+    qv = ld_any(p.proj, p.proj_dtype, qo + i) * p.q_scale;
+    bv = ld_any(p.proj, p.proj_dtype, ko + i) * p.key_scale;
+    const int c = head * p.dim + i, hd = p.H * p.dim;
+    float z = p.gate_bias[c];
+    for (int r = 0; r < p.rank; ++r) z = fmaf(p.gate_map[(size_t)r * hd + c], ld_any(p.proj, p.proj_dtype, rowp + p.low_off + r), z);
+    av = sigmoid_power(z, p.power);
   } else {
     const float rq = ld_any(p.proj, p.proj_dtype, qo + i);
     qv = rq / (1.f + expf(-rq));
@@ -97,7 +122,7 @@ __device__ __forceinline__ void transform(const RecurrenceArgs& p, int token, in
   }
 }
 
-// ready[t][0] = q, [1] = b, [2] = a (FORGET_GATE only), each [H * dim]
+// ready[t][0] = q, [1] = b, [2] = a (FORGET_GATE and KEY_DECAY), each [H * dim]
 __global__ void __launch_bounds__(256) recurrence_prepare_kernel(const RecurrenceArgs p, int T) {
   const int hd = p.H * p.dim, planes = p.mode == FORGET_GATE ? 3 : 2;
   const long n = (long)T * hd;
@@ -113,6 +138,38 @@ __global__ void __launch_bounds__(256) recurrence_prepare_kernel(const Recurrenc
   }
 }
 
+// The same for KEY_DECAY: a block takes LOW_TOKENS tokens and 256 channels, so that a row of the map
+// is read once for all of its tokens (the same chain of sums as in `transform`).
+constexpr int LOW_TOKENS = 8;
+__global__ void __launch_bounds__(256) key_decay_prepare_kernel(const RecurrenceArgs p, int T) {
+  extern __shared__ float low[];  // [LOW_TOKENS][rank]
+  const int hd = p.H * p.dim, t0 = blockIdx.x * LOW_TOKENS, n = min(LOW_TOKENS, T - t0);
+  for (int i = threadIdx.x; i < LOW_TOKENS * p.rank; i += blockDim.x) {
+    const int k = i / p.rank;
+    low[i] = k < n ? ld_any(p.proj, p.proj_dtype, (size_t)(t0 + k) * p.ld + p.low_off + i % p.rank) : 0.f;
+  }
+  __syncthreads();
+  const int c = blockIdx.y * blockDim.x + threadIdx.x;
+  if (c >= hd) return;
+  float z[LOW_TOKENS];
+#pragma unroll
+  for (int k = 0; k < LOW_TOKENS; ++k) z[k] = p.gate_bias[c];
+  for (int r = 0; r < p.rank; ++r) {
+    const float m = p.gate_map[(size_t)r * hd + c];
+#pragma unroll
+    for (int k = 0; k < LOW_TOKENS; ++k) z[k] = fmaf(m, low[k * p.rank + r], z[k]);
+  }
+#pragma unroll
+  for (int k = 0; k < LOW_TOKENS; ++k) {
+    if (k >= n || p.positions[t0 + k] < 0) continue;
+    const size_t rowp = (size_t)(t0 + k) * p.ld;
+    float* dst = p.ready + (size_t)(t0 + k) * 3 * hd + c;
+    dst[0] = ld_any(p.proj, p.proj_dtype, rowp + p.q_off + c) * p.q_scale;
+    dst[hd] = ld_any(p.proj, p.proj_dtype, rowp + p.k_off + c) * p.key_scale;
+    dst[2 * hd] = sigmoid_power(z[k], p.power);
+  }
+}
+
 __device__ __forceinline__ void cp_async4(float* smem, const float* gmem) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem));
 }
@@ -121,8 +178,8 @@ __device__ __forceinline__ void cp_async16(float* smem, const float* gmem) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem));
 }
 
-// ROWS: state rows a thread holds; TPR: tokens per staging round
-template <int ROWS, int TPR>
+// ROWS: state rows a thread holds; TPR: tokens per staging round; KIND: what a_t is
+template <int ROWS, int TPR, int KIND>
 __global__ void __launch_bounds__(THREADS)
 linear_recurrence_kernel(const RecurrenceArgs p) {
   extern __shared__ float smem[];
@@ -136,40 +193,69 @@ linear_recurrence_kernel(const RecurrenceArgs p) {
   const int dpad = p.slices * ROWS;  // state rows covered by the threads of a column (>= dim)
   constexpr int R = TPR;
   const int C = p.cols_per_block;
-  const bool gate = p.mode == FORGET_GATE;
-  const int planes = gate ? 3 : 2;
-  // one staging buffer: [planes][R][dpad] then v [R][C]; two of them when rounds arrive by cp.async
-  const int buf_floats = planes * R * dpad + R * C;
-  float* os = smem + (p.ready ? 2 : 1) * buf_floats;  // [R][C]
+  constexpr bool gate = KIND == VECTOR_DECAY, per_token = KIND == TOKEN_DECAY;
+  constexpr int planes = gate ? 3 : 2;
+  // one staging buffer: [planes][R][dpad], v [R][C], per-token numbers [2][R]; two of them when rounds
+  // arrive by cp.async
+  const bool streamed = per_token || p.ready != nullptr;
+  const int buf_floats = planes * R * dpad + R * C + (per_token ? 2 * R : 0);
+  float* os = smem + (streamed ? 2 : 1) * buf_floats;  // [R][C]
+  // row k of this thread's ROWS: four neighbours, then the next four behind all the slices' first fours
+  auto row_of = [&](int k) { return (k >> 2) * (p.slices * 4) + slice * 4 + (k & 3); };
 
   float* sp = p.state + (((size_t)p.state_slot[seq] * p.H + head) * p.dim) * p.vdim;
   float S[ROWS];
 #pragma unroll
   for (int k = 0; k < ROWS; ++k) {
-    const int i = slice + p.slices * k;
+    const int i = row_of(k);
     S[k] = (col_ok && i < p.dim) ? sp[(size_t)i * p.vdim + col] : 0.f;
   }
-  const float decay = gate ? 0.f : p.decay[head];
+  const float decay = KIND == SCALAR_DECAY ? p.decay[head] : 0.f;
+  const float skip = per_token ? p.skip[head] : 0.f;
   const int hd = p.H * p.dim;
 
   // rows beyond dim stay zero in every buffer: they are written here once and never again
   if (dpad > p.dim)
-    for (int idx = tid; idx < (p.ready ? 2 : 1) * buf_floats; idx += THREADS) smem[idx] = 0.f;
+    for (int idx = tid; idx < (streamed ? 2 : 1) * buf_floats; idx += THREADS) smem[idx] = 0.f;
   __syncthreads();
 
   // rows of 16-byte pieces where every address allows it, single floats otherwise
-  const bool wide = p.dim % 4 == 0 && (((uintptr_t)p.ready) & 15) == 0;
+  const float* rows = reinterpret_cast<const float*>(p.proj);
+  const bool whole = p.ld % 4 == 0 && (((uintptr_t)rows) & 15) == 0;
+  const bool wide = p.dim % 4 == 0 && (per_token ? whole && p.q_off % 4 == 0 && p.k_off % 4 == 0 : (((uintptr_t)p.ready) & 15) == 0);
+  // values that need no arithmetic before the recurrence arrive by cp.async too
+  const bool v_async = p.proj_dtype == DSP_F32 && p.act == 0;
+  const bool v_wide = whole && p.v_off % 4 == 0 && p.vdim % 4 == 0 && C % 4 == 0;
+  const int group0 = (head / p.heads_per_group) * p.dim;
   auto stage_async = [&](int base, float* buf) {
     const int n = min(R, t1 - base);
     for (int pl = 0; pl < planes; ++pl)
       for (int r = tid >> 5; r < n; r += THREADS / 32) {
         float* dst = buf + (pl * R + r) * dpad;
-        const float* src = p.ready + ((size_t)(base + r) * planes + pl) * hd + head * p.dim;
+        const float* src = per_token ? rows + (size_t)(base + r) * p.ld + (pl == 0 ? p.q_off : p.k_off) + group0
+                                     : p.ready + ((size_t)(base + r) * planes + pl) * hd + head * p.dim;
         if (wide)
           for (int i = (tid & 31) * 4; i < p.dim; i += 128) cp_async16(dst + i, src + i);
         else
           for (int i = tid & 31; i < p.dim; i += 32) cp_async4(dst + i, src + i);
       }
+    if (v_async) {
+      float* vs = buf + planes * R * dpad;
+      const float* src = rows + p.v_off + (size_t)head * p.vdim;
+      if (v_wide) {
+        for (int idx = tid; idx < n * (C / 4); idx += THREADS) {
+          const int r = idx / (C / 4), cl = (idx % (C / 4)) * 4, c = blockIdx.x * C + cl;
+          if (c < p.vdim) cp_async16(vs + r * C + cl, src + (size_t)(base + r) * p.ld + c);
+        }
+      } else {
+        for (int idx = tid; idx < n * C; idx += THREADS) {
+          const int r = idx / C, c = blockIdx.x * C + idx % C;
+          if (c < p.vdim) cp_async4(vs + idx, src + (size_t)(base + r) * p.ld + c);
+        }
+      }
+    }
+    if (per_token && tid < 2 * n)
+      cp_async4(buf + planes * R * dpad + R * C + (tid & 1) * R + (tid >> 1), p.steps + ((size_t)(base + (tid >> 1)) * 2 + (tid & 1)) * p.H + head);
     asm volatile("cp.async.commit_group;\n");
   };
   auto stage_values = [&](int base, float* buf) {
@@ -183,17 +269,18 @@ linear_recurrence_kernel(const RecurrenceArgs p) {
     }
   };
 
-  if (p.ready) stage_async(t0, smem);
+  if (streamed) stage_async(t0, smem);
   int turn = 0;
   for (int base = t0; base < t1; base += R, turn ^= 1) {
     const int n = min(R, t1 - base);
-    float* buf = smem + (p.ready ? turn : 0) * buf_floats;
+    float* buf = smem + (streamed ? turn : 0) * buf_floats;
     float* qs = buf;
     float* bs = buf + R * dpad;
     float* as = buf + 2 * R * dpad;
     float* vs = buf + planes * R * dpad;
-    if (p.ready) {
-      stage_values(base, buf);
+    const float* steps = vs + R * C;
+    if (streamed) {
+      if (!v_async) stage_values(base, buf);
       if (base + R < t1) {
         stage_async(base + R, smem + (turn ^ 1) * buf_floats);
         asm volatile("cp.async.wait_group 1;\n");
@@ -213,30 +300,31 @@ linear_recurrence_kernel(const RecurrenceArgs p) {
     }
     __syncthreads();
     auto one_token = [&](int r) {
-      const float v = vs[r * C + col_local];
-      const float* qr = qs + r * dpad + slice;
-      const float* br = bs + r * dpad + slice;
+      const float v = vs[r * C + col_local] * (per_token ? steps[r] : 1.f);
+      const float a_all = per_token ? steps[R + r] : decay;
+      const float* qr = qs + r * dpad + slice * 4;
+      const float* br = bs + r * dpad + slice * 4;
+      const float* ar = as + r * dpad + slice * 4;
       float acc0 = 0.f, acc1 = 0.f;
-      if (gate) {
-        const float* ar = as + r * dpad + slice;
 #pragma unroll
-        for (int k = 0; k < ROWS; k += 2) {
-          S[k] = fmaf(ar[p.slices * k], S[k], br[p.slices * k] * v);
-          acc0 = fmaf(S[k], qr[p.slices * k], acc0);
-          S[k + 1] = fmaf(ar[p.slices * (k + 1)], S[k + 1], br[p.slices * (k + 1)] * v);
-          acc1 = fmaf(S[k + 1], qr[p.slices * (k + 1)], acc1);
-        }
-      } else {
-#pragma unroll
-        for (int k = 0; k < ROWS; k += 2) {
-          S[k] = fmaf(decay, S[k], br[p.slices * k] * v);
-          acc0 = fmaf(S[k], qr[p.slices * k], acc0);
-          S[k + 1] = fmaf(decay, S[k + 1], br[p.slices * (k + 1)] * v);
-          acc1 = fmaf(S[k + 1], qr[p.slices * (k + 1)], acc1);
-        }
+      for (int k = 0; k < ROWS; k += 4) {
+        const int at = p.slices * k;
+        const float4 q4 = *reinterpret_cast<const float4*>(qr + at), b4 = *reinterpret_cast<const float4*>(br + at);
+        float4 a4 = make_float4(a_all, a_all, a_all, a_all);
+        if (gate) a4 = *reinterpret_cast<const float4*>(ar + at);
+        S[k] = fmaf(a4.x, S[k], b4.x * v);
+        acc0 = fmaf(S[k], q4.x, acc0);
+        S[k + 1] = fmaf(a4.y, S[k + 1], b4.y * v);
+        acc1 = fmaf(S[k + 1], q4.y, acc1);
+        S[k + 2] = fmaf(a4.z, S[k + 2], b4.z * v);
+        acc0 = fmaf(S[k + 2], q4.z, acc0);
+        S[k + 3] = fmaf(a4.w, S[k + 3], b4.w * v);
+        acc1 = fmaf(S[k + 3], q4.w, acc1);
       }
       return acc0 + acc1;
     };
+    // what goes out beside S^T q (read here, before the buffers turn)
+    auto direct = [&](int r) { return per_token ? skip * vs[r * C + col_local] : 0.f; };
     if (n == R) {
       // a full round: the tokens' partial outputs first, then their reductions over the slices
       // side by side (the shuffles of one token do not wait for another's)
@@ -251,13 +339,13 @@ linear_recurrence_kernel(const RecurrenceArgs p) {
         }
       if (slice == 0) {
 #pragma unroll
-        for (int r = 0; r < R; ++r) os[r * C + col_local] = acc[r];
+        for (int r = 0; r < R; ++r) os[r * C + col_local] = acc[r] + direct(r);
       }
     } else {
       for (int r = 0; r < n; ++r) {
         float acc = one_token(r);
         for (int o = 1; o < p.slices; o <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-        if (slice == 0) os[r * C + col_local] = acc;
+        if (slice == 0) os[r * C + col_local] = acc + direct(r);
       }
     }
     __syncthreads();
@@ -268,36 +356,41 @@ linear_recurrence_kernel(const RecurrenceArgs p) {
   }
 #pragma unroll
   for (int k = 0; k < ROWS; ++k) {
-    const int i = slice + p.slices * k;
+    const int i = row_of(k);
     if (col_ok && i < p.dim) sp[(size_t)i * p.vdim + col] = S[k];
   }
 }
 
-template <int ROWS, int TPR>
-int launch(const RecurrenceArgs& a, int S, size_t smem, cudaStream_t stream) {
+template <int ROWS, int TPR, int KIND>
+int launch_kind(const RecurrenceArgs& a, int S, size_t smem, cudaStream_t stream) {
   static size_t configured = 48 * 1024;
   if (smem > configured) {
-    DSP_CUDA(cudaFuncSetAttribute(linear_recurrence_kernel<ROWS, TPR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    DSP_CUDA(cudaFuncSetAttribute(linear_recurrence_kernel<ROWS, TPR, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = smem;
   }
   dim3 grid((a.vdim + a.cols_per_block - 1) / a.cols_per_block, a.H, S);
-  linear_recurrence_kernel<ROWS, TPR><<<grid, THREADS, smem, stream>>>(a);
+  linear_recurrence_kernel<ROWS, TPR, KIND><<<grid, THREADS, smem, stream>>>(a);
   DSP_CHECK_LAUNCH("dsp_linear_recurrence");
   return 0;
 }
+
+template <int ROWS, int TPR>
+int launch(const RecurrenceArgs& a, int S, size_t smem, cudaStream_t stream) {
+  if (a.mode == STEP_DECAY) return launch_kind<ROWS, TPR, TOKEN_DECAY>(a, S, smem, stream);
+  if (a.mode == FIXED_DECAY) return launch_kind<ROWS, TPR, SCALAR_DECAY>(a, S, smem, stream);
+  return launch_kind<ROWS, TPR, VECTOR_DECAY>(a, S, smem, stream);
+}
 }  // namespace
 
-// Floats of scratch the two-kernel form needs for T tokens (0: mode unknown).
-extern "C" long dsp_linear_recurrence_scratch(int mode, int H, int dim, long T) {
-  return (long)(mode == FORGET_GATE ? 3 : 2) * H * dim * T;
-}
-
-// scratch: null (one kernel, tokens transformed as they are staged) or room for
-// dsp_linear_recurrence_scratch floats (a first kernel transforms every token, the recurrence streams).
+// scratch: null (one kernel, tokens transformed as they are staged) or room for [T, planes, H * dim]
+// floats, planes = 2 with one decay for all rows, else 3 (a first kernel transforms every token, the
+// recurrence streams); STEP_DECAY takes none.
 extern "C" int dsp_linear_recurrence(const void* proj, int proj_dtype, long ld, int q_off, int k_off,
                                      int v_off, int mode, int H, int dim, int vdim, const float* decay,
                                      const float* inv_freq, int rot, float key_scale, int act,
-                                     const float* gate_bias, const float* lower, float* state,
+                                     const float* gate_bias, const float* lower,
+                                     const float* gate_map, int low_off, int rank, float q_scale, float power,
+                                     const float* steps, const float* skip, int heads_per_group, float* state,
                                      const int* state_slot, const int* q_start, const int* positions,
                                      float* out, long ldo, int S, int T, float* scratch, cudaStream_t stream) {
   if (S == 0 || T == 0) return 0;
@@ -310,6 +403,11 @@ extern "C" int dsp_linear_recurrence(const void* proj, int proj_dtype, long ld, 
     DSP_REQUIRE(act == 0 || act == 1, "dsp_linear_recurrence: unknown activation %d", act);
   } else if (mode == FORGET_GATE) {
     DSP_REQUIRE(gate_bias && lower, "dsp_linear_recurrence: no gate bias or lower bound");
+  } else if (mode == KEY_DECAY) {
+    DSP_REQUIRE(gate_bias && gate_map && rank > 0 && rank <= 1024, "dsp_linear_recurrence: no decay map or bias, or rank %d outside 1..1024", rank);
+  } else if (mode == STEP_DECAY) {
+    DSP_REQUIRE(steps && skip && proj_dtype == DSP_F32 && !scratch, "dsp_linear_recurrence: no step sizes, or rows that are not floats");
+    DSP_REQUIRE(heads_per_group > 0 && H % heads_per_group == 0, "dsp_linear_recurrence: %d heads in groups of %d", H, heads_per_group);
   } else {
     DSP_REQUIRE(false, "dsp_linear_recurrence: unknown mode %d", mode);
   }
@@ -319,6 +417,8 @@ extern "C" int dsp_linear_recurrence(const void* proj, int proj_dtype, long ld, 
   a.H = H; a.dim = dim; a.vdim = vdim;
   a.decay = decay; a.inv_freq = inv_freq; a.rot = rot; a.key_scale = key_scale; a.act = mode == FIXED_DECAY ? act : 0;
   a.gate_bias = gate_bias; a.lower = lower;
+  a.gate_map = gate_map; a.low_off = low_off; a.rank = rank; a.q_scale = q_scale; a.power = power;
+  a.steps = steps; a.skip = skip; a.heads_per_group = mode == STEP_DECAY ? heads_per_group : 1;
   a.state = state; a.state_slot = state_slot; a.q_start = q_start; a.positions = positions;
   a.out = out; a.ldo = ldo; a.ready = scratch;
   // threads per column: as many as bring a thread's state rows down to 8 (a power of two, at
@@ -331,10 +431,17 @@ extern "C" int dsp_linear_recurrence(const void* proj, int proj_dtype, long ld, 
   const int R = rows <= 8 ? 8 : (rows <= 16 ? 16 : 32);
   const int dpad = slices * R;
   a.tokens_per_round = dpad <= 256 ? 16 : 8;
-  const int planes = mode == FORGET_GATE ? 3 : 2;
-  const size_t buf = (size_t)planes * a.tokens_per_round * dpad + (size_t)a.tokens_per_round * a.cols_per_block;
-  const size_t smem = sizeof(float) * ((scratch ? 2 : 1) * buf + (size_t)a.tokens_per_round * a.cols_per_block);
-  if (scratch) {
+  const int planes = mode == FORGET_GATE || mode == KEY_DECAY ? 3 : 2;
+  const size_t buf = (size_t)planes * a.tokens_per_round * dpad + (size_t)a.tokens_per_round * a.cols_per_block +
+                     (mode == STEP_DECAY ? 2 * a.tokens_per_round : 0);
+  const size_t smem = sizeof(float) * ((scratch || mode == STEP_DECAY ? 2 : 1) * buf + (size_t)a.tokens_per_round * a.cols_per_block);
+  DSP_REQUIRE(smem <= 227 * 1024, "dsp_linear_recurrence: state rows of %d do not fit shared memory", dim);
+  if (scratch && mode == KEY_DECAY) {
+    const unsigned tiles = (unsigned)((H * dim + 255) / 256);
+    DSP_REQUIRE(tiles <= 65535, "dsp_linear_recurrence: %d heads of %d are too many", H, dim);
+    key_decay_prepare_kernel<<<dim3((T + LOW_TOKENS - 1) / LOW_TOKENS, tiles), 256, sizeof(float) * LOW_TOKENS * rank, stream>>>(a, T);
+    DSP_CHECK_LAUNCH("dsp_linear_recurrence (first kernel)");
+  } else if (scratch) {
     const long n = (long)T * H * dim;
     const int sms = dsp_num_sms();
     const long want = (n + 255) / 256, cap = (long)(sms > 0 ? sms : 148) * 8;

@@ -3,7 +3,9 @@
 // tiles and blocks beyond the real number leave at once, so a step can be captured in a graph).
 //
 //   dsp_moe_route    scores = softmax(W_router h) over all experts in 32-bit (W_router float, h of
-//                    either type), or with `score_kind` 1 the sigmoid of every logit; experts form `groups` equal runs of neighbours, a group's score
+//                    either type), or with `score_kind` 1 the sigmoid of every logit, or with 2 a softmax over
+//                    the chosen experts' logits only (groups and experts are ranked by the logits); `bias`
+//                    (float, optional) is added to the logits; experts form `groups` equal runs of neighbours, a group's score
 //                    is its largest score, only experts of the `keep` best groups can be chosen;
 //                    the `top` largest of those are the token's experts, their scores its weights
 //                    (not renormalised).  Equal scores: the lower index wins.  One block per token.
@@ -69,7 +71,8 @@ __device__ __forceinline__ Best warp_best(Best b) {
 
 // (two blocks of 1,024 threads an SM: 32 registers a thread, so that prompts' blocks of 16 warps fit four an SM)
 __global__ void __launch_bounds__(1024, 2)
-moe_route_kernel(const void* __restrict__ h, int h_dtype, long ldh, const float* __restrict__ w, int T, int W, int E,
+moe_route_kernel(const void* __restrict__ h, int h_dtype, long ldh, const float* __restrict__ w,
+                 const float* __restrict__ bias, int T, int W, int E,
                  int groups, int keep, int top, int score_kind, int group_kind, int normalize, float weight_scale,
                  int extra, float* __restrict__ extra_out, int* __restrict__ ids, float* __restrict__ wts) {
   extern __shared__ float sm[];
@@ -96,7 +99,7 @@ moe_route_kernel(const void* __restrict__ h, int h_dtype, long ldh, const float*
     }
     for (; i < W; i += 32) a0 = fmaf(we[i], hs[i], a0);
     const float acc = warp_sum((a0 + a1) + (a2 + a3));
-    if (lane == 0) sc[e] = acc;
+    if (lane == 0) sc[e] = bias ? acc + bias[e] : acc;
   }
   __syncthreads();
   if (warp != 0) return;
@@ -111,7 +114,7 @@ moe_route_kernel(const void* __restrict__ h, int h_dtype, long ldh, const float*
   // sigmoid scores are chosen by their logits: the order is the same, and two logits whose sigmoids
   // both round to 1 still differ
   for (int e = lane; e < E; e += 32) {
-    if (score_kind != 1) sc[e] = expf(sc[e] - mx) / sum;
+    if (score_kind == 0) sc[e] = expf(sc[e] - mx) / sum;
     ok[e] = 0.f;
   }
   __syncwarp();
@@ -189,6 +192,8 @@ moe_route_kernel(const void* __restrict__ h, int h_dtype, long ldh, const float*
       if (lane + 32 * k == bi) whole[k] = INT_MIN;
     __syncwarp();
   }
+  // (score_kind 2: the first winner has the largest logit of the open groups, every weight is relative to it)
+  float first = 0.f;
   // every lane holds each round's winner: the weights' sum is formed in registers (ascending r), the
   // weights wait in shared memory (the token's row is no longer needed) and go out once, scaled
   float wsum = 0.f;
@@ -196,7 +201,8 @@ moe_route_kernel(const void* __restrict__ h, int h_dtype, long ldh, const float*
     Best b = {-INFINITY, -1};
     for (int e = lane; e < E; e += 32) b = better(b, Best{sc[e], ok[e] > 0.f ? e : -1});
     b = warp_best(b);
-    const float wr = b.i < 0 ? 0.f : score_kind == 1 ? 1.f / (1.f + expf(-b.v)) : b.v;
+    if (r == 0) first = b.v;
+    const float wr = b.i < 0 ? 0.f : score_kind == 1 ? 1.f / (1.f + expf(-b.v)) : score_kind == 2 ? expf(b.v - first) : b.v;
     wsum += wr;
     if (lane == 0) {
       ids[t * top + r] = b.i;
@@ -205,7 +211,7 @@ moe_route_kernel(const void* __restrict__ h, int h_dtype, long ldh, const float*
     }
     __syncwarp();
   }
-  const float f = normalize ? weight_scale / (wsum + 1e-20f) : 1.f;
+  const float f = score_kind == 2 ? weight_scale / wsum : normalize ? weight_scale / (wsum + 1e-20f) : 1.f;
   for (int r = lane; r < top; r += 32) wts[t * top + r] = hs[r] * f;
 }
 
@@ -474,11 +480,11 @@ moe_combine_kernel(const float* __restrict__ P, long ldp, const float* __restric
 // Rows of a tile of dsp_moe_product: the tensor-core kernel's (bfloat16) or the 32-bit kernel's.
 extern "C" int dsp_moe_tile_rows(int tensor_cores) { return tensor_cores == 2 ? MMA_ROWS_WIDE : tensor_cores ? MMA_ROWS : TILE_ROWS; }
 
-extern "C" int dsp_moe_route(const void* h, int h_dtype, long ldh, const float* w, int T, int W, int E, int groups,
-                             int keep, int top, int score_kind, int group_kind, int normalize, float weight_scale,
+extern "C" int dsp_moe_route(const void* h, int h_dtype, long ldh, const float* w, const float* bias, int T, int W,
+                             int E, int groups, int keep, int top, int score_kind, int group_kind, int normalize, float weight_scale,
                              int extra, float* extra_out, int* ids, float* wts, cudaStream_t stream) {
   if (T == 0) return 0;
-  DSP_REQUIRE(score_kind == 0 || score_kind == 1, "dsp_moe_route: unknown score kind %d", score_kind);
+  DSP_REQUIRE(score_kind >= 0 && score_kind <= 2, "dsp_moe_route: unknown score kind %d", score_kind);
   DSP_REQUIRE(h && w && ids && wts, "dsp_moe_route: missing operand");
   DSP_REQUIRE(top <= W, "dsp_moe_route: top=%d exceeds the row's width %d", top, W);
   DSP_REQUIRE(groups <= 32 * GROUPS_PER_LANE, "dsp_moe_route: %d groups are more than the router ranks (%d)", groups,
@@ -502,7 +508,7 @@ extern "C" int dsp_moe_route(const void* h, int h_dtype, long ldh, const float* 
         break;
       }
   const unsigned threads = 32u * (unsigned)warps;
-  DSP_CUDA(launch_plain(moe_route_kernel, dim3((unsigned)T), dim3(threads), smem, stream, h, h_dtype, ldh, w, T, W, E,
+  DSP_CUDA(launch_plain(moe_route_kernel, dim3((unsigned)T), dim3(threads), smem, stream, h, h_dtype, ldh, w, bias, T, W, E,
                         groups, keep, top, score_kind, group_kind, normalize, weight_scale, extra, extra_out, ids, wts));
   DSP_CHECK_LAUNCH("dsp_moe_route");
   return 0;

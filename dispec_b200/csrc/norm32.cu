@@ -35,50 +35,56 @@ sum_norm_kernel(const void* __restrict__ x, int x_dtype, long ldx, const void* _
 }
 
 // Per (token, head): y = o / sqrt(mean(o^2) + eps) * gain[j] * act(gate[t, head, j])
-// (gain and gate optional; act is silu, or the logistic sigmoid when gate_kind is 1).
+// (gain and gate optional; act is silu, or the logistic sigmoid when gate_kind is 1).  `gain_ld` is the
+// distance between the gains of neighbouring heads (0: one gain of size dv for all of them).  With
+// `gate_first` the gate comes before the norm: g = o * act(gate), y = g / sqrt(mean(g^2) + eps) * gain[j].
 // o is float [T, H * dv]; one warp per (token, head).
+__device__ __forceinline__ float gate_act(float g, int kind) { return (kind == 1 ? 1.f : g) / (1.f + expf(-g)); }
+
 __global__ void __launch_bounds__(128)
-head_norm_gate_kernel(const float* __restrict__ o, long ldo, const float* __restrict__ gain,
+head_norm_gate_kernel(const float* __restrict__ o, long ldo, const float* __restrict__ gain, int gain_ld,
                       const void* __restrict__ gate, int g_dtype, long ldg, void* __restrict__ y,
-                      int y_dtype, long ldy, int T, int H, int dv, float eps, int gate_kind) {
+                      int y_dtype, long ldy, int T, int H, int dv, float eps, int gate_kind, int gate_first) {
   const int lane = threadIdx.x & 31;
   const long pair = (long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (pair >= (long)T * H) return;
   const int t = (int)(pair / H), h = (int)(pair % H);
   const float* row = o + (size_t)t * ldo + (size_t)h * dv;
+  const size_t g0 = (size_t)t * ldg + (size_t)h * dv;
   float ss = 0.f;
-  for (int j = lane; j < dv; j += 32) ss = fmaf(row[j], row[j], ss);
+  for (int j = lane; j < dv; j += 32) {
+    const float v = gate_first ? row[j] * gate_act(ld_any(gate, g_dtype, g0 + j), gate_kind) : row[j];
+    ss = fmaf(v, v, ss);
+  }
   ss = warp_sum(ss);
   const float inv = 1.f / sqrtf(ss / (float)dv + eps);
   for (int j = lane; j < dv; j += 32) {
     float v = row[j] * inv;
-    if (gain) v *= gain[j];
-    if (gate) {
-      const float g = ld_any(gate, g_dtype, (size_t)t * ldg + (size_t)h * dv + j);
-      v *= (gate_kind == 1 ? 1.f : g) / (1.f + expf(-g));
-    }
+    if (gain) v *= gain[(size_t)h * gain_ld + j];
+    if (gate) v *= gate_act(ld_any(gate, g_dtype, g0 + j), gate_kind);
     st_any(y, y_dtype, (size_t)t * ldy + (size_t)h * dv + j, v);
   }
 }
 
 // The same for wide heads (a "head" may be the whole row): one block per (token, head).
 __global__ void __launch_bounds__(256)
-head_norm_gate_wide_kernel(const float* __restrict__ o, long ldo, const float* __restrict__ gain,
+head_norm_gate_wide_kernel(const float* __restrict__ o, long ldo, const float* __restrict__ gain, int gain_ld,
                            const void* __restrict__ gate, int g_dtype, long ldg, void* __restrict__ y,
-                           int y_dtype, long ldy, int H, int dv, float eps, int gate_kind) {
+                           int y_dtype, long ldy, int H, int dv, float eps, int gate_kind, int gate_first) {
   __shared__ float scratch[32];
   const int t = blockIdx.x / H, h = blockIdx.x % H;
   const float* row = o + (size_t)t * ldo + (size_t)h * dv;
+  const size_t g0 = (size_t)t * ldg + (size_t)h * dv;
   float ss = 0.f;
-  for (int j = threadIdx.x; j < dv; j += blockDim.x) ss = fmaf(row[j], row[j], ss);
+  for (int j = threadIdx.x; j < dv; j += blockDim.x) {
+    const float v = gate_first ? row[j] * gate_act(ld_any(gate, g_dtype, g0 + j), gate_kind) : row[j];
+    ss = fmaf(v, v, ss);
+  }
   const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)dv + eps);
   for (int j = threadIdx.x; j < dv; j += blockDim.x) {
     float v = row[j] * inv;
-    if (gain) v *= gain[j];
-    if (gate) {
-      const float g = ld_any(gate, g_dtype, (size_t)t * ldg + (size_t)h * dv + j);
-      v *= (gate_kind == 1 ? 1.f : g) / (1.f + expf(-g));
-    }
+    if (gain) v *= gain[(size_t)h * gain_ld + j];
+    if (gate) v *= gate_act(ld_any(gate, g_dtype, g0 + j), gate_kind);
     st_any(y, y_dtype, (size_t)t * ldy + (size_t)h * dv + j, v);
   }
 }
@@ -119,11 +125,11 @@ xielu_kernel(const void* __restrict__ z, int z_dtype, long ldz, const float* __r
   }
 }
 
-// Layer norm with a gain and no bias: y = (x - mean) / sqrt(var + eps) * w, var the mean of the
+// Layer norm with a gain and an optional bias: y = (x - mean) / sqrt(var + eps) * w + b, var the mean of the
 // squared deviations (two passes over the row held in shared memory).  `rows` gathers input rows.
 __global__ void __launch_bounds__(256)
-layer_norm_kernel(const void* __restrict__ x, int x_dtype, long ldx, const float* __restrict__ w, float eps,
-                  const int* __restrict__ rows, void* __restrict__ y, int y_dtype, long ldy, int width) {
+layer_norm_kernel(const void* __restrict__ x, int x_dtype, long ldx, const float* __restrict__ w,
+                  const float* __restrict__ b, float eps, const int* __restrict__ rows, void* __restrict__ y, int y_dtype, long ldy, int width) {
   extern __shared__ float row[];
   __shared__ float scratch[32];
   const int r = blockIdx.x;
@@ -142,24 +148,24 @@ layer_norm_kernel(const void* __restrict__ x, int x_dtype, long ldx, const float
   }
   const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
   for (int i = threadIdx.x; i < width; i += blockDim.x)
-    st_any(y, y_dtype, (size_t)r * ldy + i, (row[i] - mean) * inv * w[i]);
+    st_any(y, y_dtype, (size_t)r * ldy + i, fmaf((row[i] - mean) * inv, w[i], b ? b[i] : 0.f));
 }
 
 // One update of a 32-bit residual stream and, optionally, what the next reader wants of it:
 //
 //     x <- x + d,   d = y * scale[i] * sigmoid(gate)        (gate given: a gated, scaled sublayer)
 //                   d = y / sqrt(mean(y^2) + eps) * rms_w   (rms_w given: an RMS-normed addend)
-//                   d = y                                   (neither; y may be missing: d = 0)
+//                   d = y * y_scale                         (neither; y may be missing: d = 0)
 //     and d += bias[i] when a row `bias` is given (the same for every row),
-//     out = layer_norm(x) * norm_w  (norm_w given; with `norm_rms` the RMS norm
+//     out = layer_norm(x) * norm_w + norm_b  (norm_w given, norm_b optional; with `norm_rms` the RMS norm
 //           x / sqrt(mean(x^2) + eps) * norm_w instead)  or  x   (out given without norm_w)
 //
 // One block per row; the new row stays in shared memory between the passes.
 __global__ void __launch_bounds__(256)
 stream_update_kernel(float* __restrict__ x32, long ldx, const void* __restrict__ y, int y_dtype, long ldy,
                      const void* __restrict__ gate, int g_dtype, long ldg, const float* __restrict__ scale,
-                     const float* __restrict__ rms_w, float rms_eps, const float* __restrict__ bias,
-                     const float* __restrict__ norm_w, float norm_eps, int norm_rms, void* __restrict__ out,
+                     const float* __restrict__ rms_w, float rms_eps, const float* __restrict__ bias, float y_scale,
+                     const float* __restrict__ norm_w, const float* __restrict__ norm_b, float norm_eps, int norm_rms, void* __restrict__ out,
                      int out_dtype, long ldo, int width) {
   extern __shared__ float row[];
   __shared__ float scratch[32];
@@ -181,6 +187,8 @@ stream_update_kernel(float* __restrict__ x32, long ldx, const void* __restrict__
       d *= (scale ? scale[i] : 1.f) * (1.f / (1.f + expf(-g)));
     } else if (rms_w) {
       d *= inv_rms * rms_w[i];
+    } else {
+      d *= y_scale;
     }
     if (bias) d += bias[i];
     const float v = x32[r * ldx + i] + d;
@@ -202,7 +210,7 @@ stream_update_kernel(float* __restrict__ x32, long ldx, const void* __restrict__
   }
   const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)width + norm_eps);
   for (int i = threadIdx.x; i < width; i += blockDim.x)
-    st_any(out, out_dtype, r * ldo + i, (row[i] - mean) * inv * norm_w[i]);
+    st_any(out, out_dtype, r * ldo + i, fmaf((row[i] - mean) * inv, norm_w[i], norm_b ? norm_b[i] : 0.f));
 }
 
 // Gated linear unit with clamps: row = [gates | ups]; g = min(gate, limit), u = clamp(up, -limit, limit);
@@ -352,21 +360,22 @@ extern "C" int dsp_sum_norm(const void* x, int x_dtype, long ldx, const void* de
   return 0;
 }
 
-extern "C" int dsp_head_norm_gate(const float* o, long ldo, const float* gain, const void* gate,
+extern "C" int dsp_head_norm_gate(const float* o, long ldo, const float* gain, int gain_ld, const void* gate,
                                   int g_dtype, long ldg, void* y, int y_dtype, long ldy, int T, int H,
-                                  int dv, float eps, int gate_kind, cudaStream_t stream) {
+                                  int dv, float eps, int gate_kind, int gate_first, cudaStream_t stream) {
   if (T == 0) return 0;
   DSP_REQUIRE(o && y && H > 0 && dv > 0, "dsp_head_norm_gate: missing operand");
   DSP_REQUIRE(gate_kind == 0 || gate_kind == 1, "dsp_head_norm_gate: unknown gate kind %d", gate_kind);
+  DSP_REQUIRE(!gate_first || gate, "dsp_head_norm_gate: a gate before the norm but no gate");
   const long pairs = (long)T * H;
   if (dv >= 512) {
-    DSP_CUDA(launch_plain(head_norm_gate_wide_kernel, dim3((unsigned)pairs), dim3(256), 0, stream, o, ldo, gain, gate,
-                          g_dtype, ldg, y, y_dtype, ldy, H, dv, eps, gate_kind));
+    DSP_CUDA(launch_plain(head_norm_gate_wide_kernel, dim3((unsigned)pairs), dim3(256), 0, stream, o, ldo, gain, gain_ld,
+                          gate, g_dtype, ldg, y, y_dtype, ldy, H, dv, eps, gate_kind, gate_first));
     DSP_CHECK_LAUNCH("dsp_head_norm_gate");
     return 0;
   }
   DSP_CUDA(launch_plain(head_norm_gate_kernel, dim3((unsigned)((pairs + 3) / 4)), dim3(128), 0, stream, o,
-                      ldo, gain, gate, g_dtype, ldg, y, y_dtype, ldy, T, H, dv, eps, gate_kind));
+                      ldo, gain, gain_ld, gate, g_dtype, ldg, y, y_dtype, ldy, T, H, dv, eps, gate_kind, gate_first));
   DSP_CHECK_LAUNCH("dsp_head_norm_gate");
   return 0;
 }
@@ -384,15 +393,15 @@ extern "C" int dsp_xielu(const void* z, int z_dtype, long ldz, const float* pq, 
   return 0;
 }
 
-extern "C" int dsp_layer_norm(const void* x, int x_dtype, long ldx, const float* w, float eps, const int* rows,
-                              void* y, int y_dtype, long ldy, int n_rows, int width, cudaStream_t stream) {
+extern "C" int dsp_layer_norm(const void* x, int x_dtype, long ldx, const float* w, const float* b, float eps,
+                              const int* rows, void* y, int y_dtype, long ldy, int n_rows, int width, cudaStream_t stream) {
   if (n_rows == 0) return 0;
   DSP_REQUIRE(x && w && y && width > 0, "dsp_layer_norm: missing operand");
   const size_t smem = (size_t)width * sizeof(float);
   DSP_REQUIRE(smem <= 200 * 1024, "dsp_layer_norm: a row of %d values does not fit shared memory", width);
   static size_t configured = 48 * 1024;
   DSP_REQUIRE(row_smem((const void*)layer_norm_kernel, smem, &configured) == 0, "dsp_layer_norm: shared memory opt-in failed");
-  DSP_CUDA(launch_plain(layer_norm_kernel, dim3(n_rows), dim3(256), smem, stream, x, x_dtype, ldx, w, eps, rows, y,
+  DSP_CUDA(launch_plain(layer_norm_kernel, dim3(n_rows), dim3(256), smem, stream, x, x_dtype, ldx, w, b, eps, rows, y,
                         y_dtype, ldy, width));
   DSP_CHECK_LAUNCH("dsp_layer_norm");
   return 0;
@@ -400,8 +409,8 @@ extern "C" int dsp_layer_norm(const void* x, int x_dtype, long ldx, const float*
 
 extern "C" int dsp_stream_update(float* x32, long ldx, const void* y, int y_dtype, long ldy, const void* gate,
                                  int g_dtype, long ldg, const float* scale, const float* rms_w, float rms_eps,
-                                 const float* bias, const float* norm_w, float norm_eps, int norm_rms, void* out,
-                                 int out_dtype, long ldo, int n_rows, int width, cudaStream_t stream) {
+                                 const float* bias, float y_scale, const float* norm_w, const float* norm_b,
+                                 float norm_eps, int norm_rms, void* out, int out_dtype, long ldo, int n_rows, int width, cudaStream_t stream) {
   if (n_rows == 0) return 0;
   DSP_REQUIRE(x32 && width > 0, "dsp_stream_update: missing operand");
   DSP_REQUIRE(y || (!gate && !rms_w), "dsp_stream_update: a gate or a norm but no addend");
@@ -411,7 +420,7 @@ extern "C" int dsp_stream_update(float* x32, long ldx, const void* y, int y_dtyp
   static size_t configured = 48 * 1024;
   DSP_REQUIRE(row_smem((const void*)stream_update_kernel, smem, &configured) == 0, "dsp_stream_update: shared memory opt-in failed");
   DSP_CUDA(launch_plain(stream_update_kernel, dim3(n_rows), dim3(256), smem, stream, x32, ldx, y, y_dtype, ldy, gate,
-                        g_dtype, ldg, scale, rms_w, rms_eps, bias, norm_w, norm_eps, norm_rms, out, out_dtype, ldo, width));
+                        g_dtype, ldg, scale, rms_w, rms_eps, bias, y_scale, norm_w, norm_b, norm_eps, norm_rms, out, out_dtype, ldo, width));
   DSP_CHECK_LAUNCH("dsp_stream_update");
   return 0;
 }

@@ -1,0 +1,215 @@
+// Short causal convolutions over time, channel by channel, with the last taps - 1 inputs of every
+// request kept in its state slot (32-bit floats, zeros at admission):
+//
+//     y_t[c] = sum_j w[j][c] * u_(t - taps + 1 + j)[c]          (w float [taps, channels])
+//
+// where u are columns of the rows of a mixer's fused projection (float or bfloat16).  Two users:
+//
+//   dsp_conv_steps             y, plus a bias, through silu, as float rows [T, channels]; and, for a state-space
+//                              recurrence, per token and head step = softplus(raw + bias) and decay =
+//                              exp(-exp(A_log) * step) as `steps` [T, 2, heads].
+//   dsp_qkv_conv_rotate_store  y over the columns [q (H x Dk) | k (G x Dk) | v (G x Dv)], then queries and keys
+//                              turned by position * inv_freq[i], pairs (2i, 2i + 1) or (i, i + rot/2), then
+//                              divided by their root mean square per head (eps inside the root, no
+//                              weight) if asked for; queries go to q_out, keys and values (times
+//                              v_scale) to the pages.
+//
+// Every token has a block (or a row of blocks) of its own: its taps come from the rows of the step, and,
+// before the first token the step brings for the request, from the state slot.  The block of that
+// first token is the only one that touches the slot: it also computes the tokens 1 .. taps - 2, which would
+// have to read it too, and then leaves the step's last taps - 1 inputs there, which it takes from
+// the projection's rows, not from other blocks.  A thread keeps to its own channels throughout, so
+// within the block nothing is ordered by barriers.  Rows with a negative position (padding of a captured
+// step) are skipped: their state slot belongs to someone else.
+#include "common.cuh"
+
+namespace {
+
+struct ConvIn {
+  const void* u;  // [T, ld], first convolved column at `off`
+  int dtype;
+  long ld;
+  int off, channels, taps;
+  const float* w;  // [taps, channels] (null: taps == 1 and y = u)
+  float* hist;     // [slots, taps - 1, channels]
+  const int* state_slot;
+  const int* q_start;
+  const int* seq_of_token;
+  const int* positions;
+};
+
+// What a block of token t does: its first local token, how many, and whether it owns the state slot.
+struct Turn {
+  int seq, first, count, n, row0;
+  bool owner;
+};
+__device__ __forceinline__ Turn turn_of(const ConvIn& c, int t) {
+  Turn r;
+  r.seq = c.seq_of_token[t];
+  r.row0 = c.q_start[r.seq];
+  r.n = c.q_start[r.seq + 1] - r.row0;
+  const int i = t - r.row0;
+  r.first = i;
+  r.owner = i == 0;
+  r.count = i == 0 ? min(r.n, max(1, c.taps - 1)) : (i < c.taps - 1 ? 0 : 1);
+  return r;
+}
+
+// input of channel c at local token j of the request's portion (negative: from the state slot)
+__device__ __forceinline__ float input_at(const ConvIn& p, const Turn& r, const float* hist, int c, int j) {
+  if (j >= 0) return ld_any(p.u, p.dtype, (size_t)(r.row0 + j) * p.ld + p.off + c);
+  return hist[(size_t)(p.taps - 1 + j) * p.channels + c];
+}
+
+__device__ __forceinline__ float conv_at(const ConvIn& p, const Turn& r, const float* hist, int c, int i) {
+  if (!p.w) return input_at(p, r, hist, c, i);
+  float acc = 0.f;
+  for (int j = 0; j < p.taps; ++j) acc = fmaf(p.w[(size_t)j * p.channels + c], input_at(p, r, hist, c, i - p.taps + 1 + j), acc);
+  return acc;
+}
+
+// leaves the portion's last taps - 1 inputs of channel c in the slot (in place: row m is written before
+// the rows behind it are, and reads rows at or behind m + n)
+__device__ __forceinline__ void keep_inputs(const ConvIn& p, const Turn& r, float* hist, int c) {
+  for (int m = 0; m < p.taps - 1; ++m)
+    hist[(size_t)m * p.channels + c] = input_at(p, r, hist, c, r.n - (p.taps - 1) + m);
+}
+
+__device__ __forceinline__ float softplus_f(float v) { return v > 20.f ? v + log1pf(expf(-v)) : log1pf(expf(v)); }
+
+constexpr int PER_THREAD = 4;
+
+__global__ void __launch_bounds__(256)
+conv_steps_kernel(const ConvIn p, const float* __restrict__ bias, float* __restrict__ out, long ldo, int step_off,
+                  int heads, const float* __restrict__ step_bias, const float* __restrict__ a_log,
+                  float* __restrict__ steps) {
+  const int t = blockIdx.x;
+  if (p.positions[t] < 0) return;
+  const Turn r = turn_of(p, t);
+  float* hist = p.hist + (size_t)p.state_slot[r.seq] * (p.taps - 1) * p.channels;
+  for (int i = r.first; i < r.first + r.count; ++i)
+#pragma unroll
+    for (int k = 0; k < PER_THREAD; ++k) {
+      const int c = (blockIdx.y * PER_THREAD + k) * 256 + threadIdx.x;
+      if (c >= p.channels) break;
+      const float v = conv_at(p, r, hist, c, i) + (bias ? bias[c] : 0.f);
+      out[(size_t)(r.row0 + i) * ldo + c] = v / (1.f + expf(-v));
+    }
+  if (r.owner)
+    for (int k = 0; k < PER_THREAD; ++k) {
+      const int c = (blockIdx.y * PER_THREAD + k) * 256 + threadIdx.x;
+      if (c < p.channels) keep_inputs(p, r, hist, c);
+    }
+  if (blockIdx.y == 0)
+    for (int h = threadIdx.x; h < heads; h += blockDim.x) {
+      const float step = softplus_f(ld_any(p.u, p.dtype, (size_t)t * p.ld + step_off + h) + step_bias[h]);
+      steps[((size_t)t * 2) * heads + h] = step;
+      steps[((size_t)t * 2 + 1) * heads + h] = expf(-expf(a_log[h]) * step);
+    }
+}
+
+__global__ void __launch_bounds__(256)
+qkv_conv_rotate_store_kernel(const ConvIn p, const int* __restrict__ page_table, int pt_stride, void* __restrict__ k_pool,
+                             void* __restrict__ v_pool, int pool_dtype, const float* __restrict__ inv_freq, int rot,
+                             int interleaved, int head_norm, float norm_eps, float v_scale, void* __restrict__ q_out,
+                             long ld_q, int H, int G, int Dk, int Dv, int page_size, int num_pages, int write_kv, int* err) {
+  extern __shared__ float row[];  // [channels] then [rot/2] cosines, [rot/2] sines
+  const int t = blockIdx.x;
+  if (p.positions[t] < 0) return;
+  const Turn r = turn_of(p, t);
+  if (r.count == 0) return;
+  float* hist = p.taps > 1 ? p.hist + (size_t)p.state_slot[r.seq] * (p.taps - 1) * p.channels : nullptr;
+  float* cs = row + p.channels;
+  const int half = rot / 2, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
+  for (int i = r.first; i < r.first + r.count; ++i) {
+    const int tok = r.row0 + i, pos = p.positions[tok];
+    for (int c = tid; c < p.channels; c += blockDim.x) row[c] = conv_at(p, r, hist, c, i);
+    for (int m = tid; m < half; m += blockDim.x) sincosf((float)pos * inv_freq[m], &cs[half + m], &cs[m]);
+    __syncthreads();
+    const int page = write_kv ? page_table[(size_t)r.seq * pt_stride + pos / page_size] : -1;
+    const bool store = write_kv && page >= 0 && page < num_pages;
+    if (write_kv && !store && tid == 0) atomicOr(err, DSP_ERR_BAD_PAGE);
+    const size_t at = (size_t)page * G * page_size + pos % page_size;  // (used only when `store`)
+    for (int h = warp; h < H + G; h += warps) {
+      float* x = row + h * Dk;
+      for (int m = lane; m < half; m += 32) {
+        const int a = interleaved ? 2 * m : m, b = interleaved ? 2 * m + 1 : m + half;
+        const float u = x[a], v = x[b], c = cs[m], s = cs[half + m];
+        x[a] = u * c - v * s;
+        x[b] = v * c + u * s;
+      }
+      __syncwarp();
+      float f = 1.f;
+      if (head_norm) {
+        float ss = 0.f;
+        for (int d = lane; d < Dk; d += 32) ss = fmaf(x[d], x[d], ss);
+        f = 1.f / sqrtf(warp_sum(ss) / (float)Dk + norm_eps);
+      }
+      if (h < H) {
+        for (int d = lane; d < Dk; d += 32) st_any(q_out, pool_dtype, (size_t)tok * ld_q + (size_t)h * Dk + d, x[d] * f);
+      } else if (store) {
+        for (int d = lane; d < Dk; d += 32) st_any(k_pool, pool_dtype, (at + (size_t)(h - H) * page_size) * Dk + d, x[d] * f);
+      }
+    }
+    if (store) {
+      const float* v = row + (H + G) * Dk;
+      for (int idx = tid; idx < G * Dv; idx += blockDim.x)
+        st_any(v_pool, pool_dtype, (at + (size_t)(idx / Dv) * page_size) * Dv + idx % Dv, v[idx] * v_scale);
+    }
+    __syncthreads();  // the row is taken again
+  }
+  if (r.owner && p.taps > 1)
+    for (int c = tid; c < p.channels; c += blockDim.x) keep_inputs(p, r, hist, c);
+}
+
+int check(const ConvIn& p, const char* name) {
+  DSP_REQUIRE(p.u && p.q_start && p.seq_of_token && p.positions && p.channels > 0, "%s: missing operand", name);
+  DSP_REQUIRE(p.taps >= 1 && (p.taps == 1 || (p.w && p.hist && p.state_slot)), "%s: %d taps without weights or state", name, p.taps);
+  return 0;
+}
+}  // namespace
+
+extern "C" int dsp_conv_steps(const void* u, int dtype, long ld, int off, int channels, int taps, const float* w,
+                              const float* bias, float* hist, const int* state_slot, const int* q_start,
+                              const int* seq_of_token, const int* positions, float* out, long ldo, int step_off, int heads,
+                              const float* step_bias, const float* a_log, float* steps, int T, cudaStream_t stream) {
+  if (T == 0) return 0;
+  const ConvIn p = {u, dtype, ld, off, channels, taps, w, hist, state_slot, q_start, seq_of_token, positions};
+  if (const int rc = check(p, "dsp_conv_steps")) return rc;
+  DSP_REQUIRE(out && w && state_slot && (heads == 0 || (step_bias && a_log && steps)), "dsp_conv_steps: missing operand");
+  const int tiles = (channels + 256 * PER_THREAD - 1) / (256 * PER_THREAD);
+  DSP_REQUIRE(tiles <= 65535, "dsp_conv_steps: %d channels are too many", channels);
+  DSP_CUDA(launch_plain(conv_steps_kernel, dim3(T, tiles), dim3(256), 0, stream, p, bias, out, ldo, step_off, heads,
+                        step_bias, a_log, steps));
+  DSP_CHECK_LAUNCH("dsp_conv_steps");
+  return 0;
+}
+
+extern "C" int dsp_qkv_conv_rotate_store(const void* u, int dtype, long ld, int taps, const float* w, float* hist,
+                                         const int* state_slot, const int* q_start, const int* seq_of_token,
+                                         const int* positions, const int* page_table, int pt_stride, void* k_pool,
+                                         void* v_pool, int pool_dtype, const float* inv_freq, int rot, int interleaved,
+                                         int head_norm, float norm_eps, float v_scale, void* q_out, long ld_q, int T, int H,
+                                         int G, int Dk, int Dv, int page_size, int num_pages, int write_kv,
+                                         cudaStream_t stream) {
+  if (T == 0) return 0;
+  DSP_REQUIRE(H > 0 && G > 0 && Dk > 0 && Dv > 0 && q_out, "dsp_qkv_conv_rotate_store: missing operand");
+  const ConvIn p = {u, dtype, ld, 0, (H + G) * Dk + G * Dv, taps, w, hist, state_slot, q_start, seq_of_token, positions};
+  if (const int rc = check(p, "dsp_qkv_conv_rotate_store")) return rc;
+  DSP_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= Dk && (rot == 0 || inv_freq), "dsp_qkv_conv_rotate_store: rot=%d for keys of %d", rot, Dk);
+  DSP_REQUIRE(!write_kv || (k_pool && v_pool && page_table && page_size > 0), "dsp_qkv_conv_rotate_store: no pools to write to");
+  int* err = dsp_device_error_ptr();
+  DSP_REQUIRE(err != nullptr, "dsp_qkv_conv_rotate_store: no device error word");
+  const size_t smem = (size_t)(p.channels + rot) * sizeof(float);
+  DSP_REQUIRE(smem <= 200 * 1024, "dsp_qkv_conv_rotate_store: rows of %d values do not fit shared memory", p.channels);
+  static size_t configured = 48 * 1024;
+  if (smem > configured) {
+    DSP_CUDA(cudaFuncSetAttribute(qkv_conv_rotate_store_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    configured = smem;
+  }
+  DSP_CUDA(launch_plain(qkv_conv_rotate_store_kernel, dim3(T), dim3(256), smem, stream, p, page_table, pt_stride, k_pool,
+                        v_pool, pool_dtype, inv_freq, rot, interleaved, head_norm, norm_eps, v_scale, q_out, ld_q, H, G, Dk,
+                        Dv, page_size, num_pages, write_kv, err));
+  DSP_CHECK_LAUNCH("dsp_qkv_conv_rotate_store");
+  return 0;
+}

@@ -65,7 +65,7 @@ class DecoderModel:
         needs: dict[int, CacheNeed] = {}
         writers: dict[int, int] = {}
         self.state_needs: list[StateNeed] = []
-        self.call_state: list[int | None] = []
+        self.call_state: list[int | tuple | None] = []
         self.call_cache: list[int | None] = []
         for idx, call in enumerate(self.schedule):
             mixer = self.layers[call.layer].mixer
@@ -86,7 +86,10 @@ class DecoderModel:
                     raise ValueError(f"schedule entry {idx} reads cache {label} before any entry wrote it")
             self.call_cache.append(label)
             sneed = mixer.state_need()
-            if sneed is not None:
+            if isinstance(sneed, tuple):
+                self.call_state.append(tuple(range(len(self.state_needs), len(self.state_needs) + len(sneed))))
+                self.state_needs.extend(sneed)
+            elif sneed is not None:
                 self.call_state.append(len(self.state_needs))
                 self.state_needs.append(sneed)
             else:
@@ -102,7 +105,7 @@ class DecoderModel:
             g = group_keys.index(need)
             self.placement[label] = CachePlacement(g, len(members[g]))
             members[g].append(label)
-        self.cache_groups = [CacheGroupSpec(tuple(k.tensors), k.window, len(m))
+        self.cache_groups = [CacheGroupSpec(tuple(k.tensors), k.window, len(m), k.keep_first)
                              for k, m in zip(group_keys, members)]
         tiles: set = set()
         for c in self.schedule:
@@ -151,7 +154,10 @@ class DecoderModel:
             label = self.call_cache[idx]
             cache = ctx.cache_view(self.placement[label], call.write) if label is not None else None
             sidx = self.call_state[idx]
-            state = ctx.state_view(sidx) if sidx is not None else None
+            if isinstance(sidx, tuple):
+                state = tuple(ctx.state_view(i) for i in sidx)
+            else:
+                state = ctx.state_view(sidx) if sidx is not None else None
             # a block may take its first norm from the product that wrote x (see PreNormBlock)
             # (not across the start of a pass: the stream changes there before the norm reads it)
             nxt = None

@@ -37,14 +37,15 @@ def paged_attention_generic(q: torch.Tensor, q_stride: int, k_pool: torch.Tensor
                             seq_of_token: torch.Tensor, out: torch.Tensor, num_heads: int,
                             num_kv_heads: int, head_dim: int, window: int, scale: float,
                             sink: bool = False, chunked: bool = False, sink_values: torch.Tensor | None = None,
-                            turn_freq: torch.Tensor | None = None) -> torch.Tensor:
+                            turn_freq: torch.Tensor | None = None, keep_first: int = 0) -> torch.Tensor:
     """32-bit arithmetic kernel, any value size up to 512 and any group size.
 
     q: element (t, h, d) at q.data_ptr + (t * q_stride + h * D + d); out: [T, H * Dv], Dv being the
     width of the value pool (it may differ from the keys' D).
     The query at absolute position p = positions[t] sees keys max(0, p-window+1)..p
     (window 0: from 0) of sequence seq_of_token[t]; with ``chunked`` the keys of its own chunk of
-    ``window`` positions, floor(p / window) * window .. p.  ``sink``: the softmax has one more key
+    ``window`` positions, floor(p / window) * window .. p; with ``keep_first`` = F also the keys
+    0..F-1.  ``sink``: the softmax has one more key
     of score 0 and no value (weights exp(s_j) / (1 + sum exp(s_j))); with ``sink_values`` (float32
     [H]) that key's score is the head's own number, unscaled.  ``turn_freq`` (float32 [Dv/2]):
     every head's result is turned back, pair (m, m + Dv/2) by -p * turn_freq[m].
@@ -55,7 +56,7 @@ def paged_attention_generic(q: torch.Tensor, q_stride: int, k_pool: torch.Tensor
     dv = v_pool.shape[3]
     assert (kvh, d) == (num_kv_heads, head_dim) and v_pool.shape[:3] == k_pool.shape[:3]
     assert k_pool.is_contiguous() and v_pool.is_contiguous() and k_pool.dtype == q.dtype == v_pool.dtype
-    assert out.is_contiguous() and out.shape == (T, num_heads * dv) and out.dtype in (q.dtype, torch.float32)
+    assert out.stride(1) == 1 and out.shape == (T, num_heads * dv) and out.dtype in (q.dtype, torch.float32)
     assert page_table.dtype == torch.int32 and page_table.stride(1) == 1
     assert positions.dtype == torch.int32 and seq_of_token.dtype == torch.int32
     _check_sink_turn(sink, sink_values, turn_freq, num_heads, dv)
@@ -63,7 +64,7 @@ def paged_attention_generic(q: torch.Tensor, q_stride: int, k_pool: torch.Tensor
         L.ptr(q), L.i64(q_stride), L.ptr(k_pool), L.ptr(v_pool), L.ptr(page_table),
         page_table.stride(0), L.ptr(positions), L.ptr(seq_of_token), L.ptr(out),
         L.i64(out.stride(0)), T, num_heads, num_kv_heads, head_dim, dv, page_size, num_pages,
-        window, int(bool(chunked) and window > 0), L.f32(scale), int(bool(sink)), L.ptr(sink_values),
+        window, int(bool(chunked) and window > 0), int(keep_first), L.f32(scale), int(bool(sink)), L.ptr(sink_values),
         L.ptr(turn_freq), L.dtype_code(q.dtype), L.dtype_code(out.dtype), L.stream_handle()))
     return out
 
@@ -400,11 +401,12 @@ def sink_choose_splits(num_single: int, num_kv_heads: int, keys: int, device=Non
 def sink_attention_tiles(q, k_pool, v_pool, page_table, q_start, ctx_len, tile_seq, tile_tok0, num_tiles, out,
                          num_heads, num_kv_heads, window, scale, sink, num_single: int = 0, splits: int = 1,
                          chunked: bool = False, sink_values: torch.Tensor | None = None,
-                         turn_freq: torch.Tensor | None = None, positions: torch.Tensor | None = None) -> torch.Tensor:
+                         turn_freq: torch.Tensor | None = None, positions: torch.Tensor | None = None,
+                         keep_first: int = 0) -> torch.Tensor:
     """The tensor-core kernel over a tile list (``tokens per tile`` = 64 // group).  The first
     ``num_single`` tiles are single tokens (the first rows of the batch): with ``splits`` > 1
     their keys are cut into that many shares, merged by the combine kernel.  ``chunked``,
-    ``sink_values``, ``turn_freq``: as in ``paged_attention_generic``; ``positions`` (of the step's
+    ``sink_values``, ``turn_freq``, ``keep_first``: as in ``paged_attention_generic``; ``positions`` (of the step's
     tokens) is needed where split results are turned back."""
     num_pages, G, page_size, dk = k_pool.shape
     dv = v_pool.shape[3]
@@ -419,7 +421,7 @@ def sink_attention_tiles(q, k_pool, v_pool, page_table, q_start, ctx_len, tile_s
         rc = fn(L.ptr(q), L.i64(q.stride(0)), L.ptr(k_pool), L.ptr(v_pool), L.ptr(page_table), page_table.stride(0),
                 L.ptr(q_start), L.ptr(ctx_len), L.ptr(tile_seq), L.ptr(tile_tok0), offset, count, L.ptr(out),
                 int(out.dtype == torch.float32), L.i64(out.stride(0)), num_heads, num_kv_heads, tpt, page_size, num_pages, window, mask_mode,
-                L.f32(scale), int(bool(sink)), L.ptr(sink_values), L.ptr(turn_freq), n_splits, L.ptr(part_o), L.ptr(part_ml), ctypes.c_void_p(_device_error_address(q.device)),
+                int(keep_first), L.f32(scale), int(bool(sink)), L.ptr(sink_values), L.ptr(turn_freq), n_splits, L.ptr(part_o), L.ptr(part_ml), ctypes.c_void_p(_device_error_address(q.device)),
                 L.stream_handle())
         L.LaunchCounter.n += 1
         if rc != 0:
@@ -446,25 +448,28 @@ def sink_attention_tiles(q, k_pool, v_pool, page_table, q_start, ctx_len, tile_s
 
 def sink_paged_attention(ctx, q: torch.Tensor, cache, out: torch.Tensor, num_heads: int, num_kv_heads: int,
                          key_dim: int, value_dim: int, window: int, scale: float, sink: bool, chunked: bool = False,
-                         sink_values: torch.Tensor | None = None, turn_freq: torch.Tensor | None = None) -> torch.Tensor:
+                         sink_values: torch.Tensor | None = None, turn_freq: torch.Tensor | None = None,
+                         keep_first: int = 0) -> torch.Tensor:
     """Attention of the step over pools whose keys and values have widths of their own, with an
     optional sink in the softmax: q [T, H * Dk] (already turned), out [T, H * Dv] (of q's type, or
     float32 for a consumer that combines heads before it rounds).  bfloat16 runs
     on the tensor-core kernel where it is built for the sizes and the batch lists its tiles;
     everything else (and float32 always) on the 32-bit kernel.  ``chunked``: ``window`` is the
     size of the chunks a position's keys come from; ``sink_values``: the sink's score per head;
-    ``turn_freq``: results are turned back by the query's position (``paged_attention_generic``)."""
+    ``turn_freq``: results are turned back by the query's position; ``keep_first``: so many first keys
+    stay visible beside the window (``paged_attention_generic``)."""
     group = num_heads // num_kv_heads
     tpt = sink_tokens_per_tile(group, key_dim, value_dim)
     if q.dtype == torch.bfloat16 and tpt is not None and tpt in ctx.attention_tiles:
         tile_seq, tile_tok0, num_tiles = ctx.attention_tiles[tpt]
-        keys = min(ctx.max_ctx_len, window) if window > 0 else ctx.max_ctx_len
+        keys = min(ctx.max_ctx_len, window + keep_first) if window > 0 else ctx.max_ctx_len
         splits = sink_choose_splits(ctx.num_decode_seqs, num_kv_heads, keys, q.device)
         return sink_attention_tiles(q, cache.key_pool, cache.value_pool, cache.page_table, ctx.q_start, ctx.ctx_len,
                                     tile_seq, tile_tok0, num_tiles, out, num_heads, num_kv_heads, window, scale, sink,
                                     num_single=ctx.num_decode_seqs, splits=splits, chunked=chunked,
-                                    sink_values=sink_values, turn_freq=turn_freq, positions=ctx.positions)
+                                    sink_values=sink_values, turn_freq=turn_freq, positions=ctx.positions,
+                                    keep_first=keep_first)
     return paged_attention_generic(q, q.stride(0), cache.key_pool, cache.value_pool, cache.page_table,
                                    ctx.positions, ctx.seq_of_token, out, num_heads, num_kv_heads, key_dim,
                                    window, scale, sink=sink, chunked=chunked, sink_values=sink_values,
-                                   turn_freq=turn_freq)
+                                   turn_freq=turn_freq, keep_first=keep_first)

@@ -62,7 +62,7 @@ class NormedRows:
         return (x is not None and x.dtype == torch.bfloat16 and M <= NORM_SPLIT_MAX_ROWS
                 and self.source.stride(1) == 1 and self.source.stride(0) % 8 == 0
                 and self.source.data_ptr() % 16 == 0 and stream_supported(M, K, x, w))
-EPI_PLAIN, EPI_SWIGLU = 0, 1
+EPI_PLAIN, EPI_SWIGLU, EPI_GEGLU = 0, 1, 2
 SWIGLU_BLOCK = 16  # gate/up rows alternate in blocks of this many for the fused epilogue
 
 
@@ -119,7 +119,7 @@ def stream_supported(M: int, K: int, x: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def gate_up_swiglu_supported(x, w: torch.Tensor) -> bool:
-    """Whether silu(gate) * up can be formed in the epilogue of the gate/up product."""
+    """Whether act(gate) * up can be formed in the epilogue of the gate/up product."""
     M, K = x.shape
     if x.dtype != torch.bfloat16 or w.shape[0] % 32:
         return False
@@ -130,8 +130,8 @@ def gate_up_swiglu_supported(x, w: torch.Tensor) -> bool:
     return tcgen05_supported(x, w)
 
 
-def linear_gate_up_swiglu(x, w_interleaved, out=None):
-    """silu(x Wg^T) * (x Wu^T) in one kernel: ``w_interleaved`` holds 16 gate rows, the 16 up
+def linear_gate_up_swiglu(x, w_interleaved, out=None, act: str = "silu"):
+    """act(x Wg^T) * (x Wu^T) in one kernel (``act`` "silu" or "gelu_tanh"): ``w_interleaved`` holds 16 gate rows, the 16 up
     rows of the same outputs, the next 16 gate rows, ...  Returns [M, N/2].  ``x``: a tensor or
     ``NormedRows``."""
     assert gate_up_swiglu_supported(x, w_interleaved)
@@ -144,9 +144,10 @@ def linear_gate_up_swiglu(x, w_interleaved, out=None):
     M, N = x.shape[0], w_interleaved.shape[0]
     if out is None:
         out = torch.empty((M, N // 2), dtype=x.dtype, device=x.device)
+    epilogue = {"silu": EPI_SWIGLU, "gelu_tanh": EPI_GEGLU}[act]
     if M > STREAM_MAX_ROWS:
-        return _tcgen05(x, w_interleaved, None, None, out, epilogue=EPI_SWIGLU)
-    return _stream(x, w_interleaved, None, None, out, epilogue=EPI_SWIGLU, norm=norm)
+        return _tcgen05(x, w_interleaved, None, None, out, epilogue=epilogue)
+    return _stream(x, w_interleaved, None, None, out, epilogue=epilogue, norm=norm)
 
 
 def _library(x, w, bias, residual, out):

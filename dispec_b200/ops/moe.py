@@ -14,27 +14,31 @@ def _lib():
 
 
 def route(h: torch.Tensor, w_router: torch.Tensor, groups: int, keep: int, top: int, score: str = "softmax",
-          group_score: str = "max", normalize: bool = False, weight_scale: float = 1.0, extra_rows: int = 0):
+          group_score: str = "max", normalize: bool = False, weight_scale: float = 1.0, extra_rows: int = 0,
+          bias: torch.Tensor | None = None):
     """h [T, W] (either type), w_router float32 [E, W] -> (ids int32 [T, top], weights float32
     [T, top]): softmax over all experts in 32-bit (``score`` "sigmoid": the sigmoid of every
     expert's logit instead, chosen by the logits, so that scores which round to the same number
-    do not tie); the ``top`` largest scores among the experts
+    do not tie; "chosen_softmax": groups and experts ranked by the logits, the weights a softmax over the
+    chosen logits only, times ``weight_scale``); the ``top`` largest scores among the experts
     of the ``keep`` groups (of ``groups`` equal runs of neighbours) with the largest best score;
     the weights are those scores.  ``group_score`` "top2_sum": a group's score is the sum of its
     two largest scores.  ``normalize``: the weights are the chosen scores divided by their sum
     (+ 1e-20), times ``weight_scale``.  ``extra_rows`` = X > 0: the last X rows of ``w_router``
-    are not experts; the sigmoids of their logits come back as a third result, float32 [T, X]."""
+    are not experts; the sigmoids of their logits come back as a third result, float32 [T, X].
+    ``bias`` (float32, one number per row of ``w_router``) is added to the logits."""
     if not (h.is_cuda and w_router.is_cuda):
         raise L.KernelError("moe.route: CUDA tensors only (there is no CPU path)")
     assert h.dim() == 2 and h.stride(1) == 1 and w_router.dtype == torch.float32 and w_router.is_contiguous()
     T, W = h.shape
     E = w_router.shape[0] - extra_rows
     assert w_router.shape == (E + extra_rows, W) and E > 0
+    assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.shape == (E + extra_rows,))
     ids = torch.empty((T, top), dtype=torch.int32, device=h.device)
     wts = torch.empty((T, top), dtype=torch.float32, device=h.device)
     extra = torch.empty((T, extra_rows), dtype=torch.float32, device=h.device) if extra_rows else None
-    L.check(_lib().dsp_moe_route(L.ptr(h), L.dtype_code(h.dtype), L.i64(h.stride(0)), L.ptr(w_router), T, W, E,
-                                 groups, keep, top, {"softmax": 0, "sigmoid": 1}[score],
+    L.check(_lib().dsp_moe_route(L.ptr(h), L.dtype_code(h.dtype), L.i64(h.stride(0)), L.ptr(w_router), L.ptr(bias), T, W, E,
+                                 groups, keep, top, {"softmax": 0, "sigmoid": 1, "chosen_softmax": 2}[score],
                                  {"max": 0, "top2_sum": 1}[group_score], int(bool(normalize)), L.f32(weight_scale),
                                  extra_rows, L.ptr(extra), L.ptr(ids), L.ptr(wts), L.stream_handle()))
     return (ids, wts, extra) if extra_rows else (ids, wts)

@@ -48,23 +48,26 @@ def sum_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, delta: torch.Ten
 
 def head_norm_gate(o: torch.Tensor, num_heads: int, eps: float, out_dtype: torch.dtype,
                    gain: torch.Tensor | None = None, gate: torch.Tensor | None = None,
-                   gate_kind: str = "silu") -> torch.Tensor:
+                   gate_kind: str = "silu", gate_first: bool = False, out: torch.Tensor | None = None) -> torch.Tensor:
     """o float32 [T, H * dv]: every head's dv values divided by their root mean square (eps inside
     the root), times ``gain`` [dv] (optional) and act(gate[t, h * dv + j]) (optional; ``gate_kind``
-    "silu" or "sigmoid").  With ``num_heads`` 1 the whole row is normed together."""
+    "silu" or "sigmoid").  With ``num_heads`` 1 the whole row is normed together.  A ``gain`` of
+    H * dv values gives every head gains of its own.  ``gate_first``: the gate multiplies o before
+    the norm.  ``out``: where the result goes (columns of a wider matrix, say)."""
     _rows2d(o, "head_norm_gate")
     assert o.dtype == torch.float32 and o.shape[1] % num_heads == 0
     T, dv = o.shape[0], o.shape[1] // num_heads
     if gain is not None:
-        assert gain.dtype == torch.float32 and gain.shape == (dv,) and gain.is_contiguous()
+        assert gain.dtype == torch.float32 and gain.shape in ((dv,), (num_heads * dv,)) and gain.is_contiguous()
     if gate is not None:
         _rows2d(gate, "head_norm_gate")
         assert gate.shape == o.shape
-    y = torch.empty((T, o.shape[1]), dtype=out_dtype, device=o.device)
+    y = out if out is not None else torch.empty((T, o.shape[1]), dtype=out_dtype, device=o.device)
+    assert y.shape == o.shape and y.dtype == out_dtype and y.stride(1) == 1 and not (gate_first and gate is None)
     L.check(L.core().dsp_head_norm_gate(
-        L.ptr(o), L.i64(o.stride(0)), L.ptr(gain), L.ptr(gate), L.dtype_code(gate.dtype) if gate is not None else 0,
+        L.ptr(o), L.i64(o.stride(0)), L.ptr(gain), dv if gain is not None and gain.shape[0] != dv else 0, L.ptr(gate), L.dtype_code(gate.dtype) if gate is not None else 0,
         L.i64(gate.stride(0) if gate is not None else 0), L.ptr(y), L.dtype_code(out_dtype), L.i64(y.stride(0)),
-        T, num_heads, dv, L.f32(eps), {"silu": 0, "sigmoid": 1}[gate_kind], L.stream_handle()))
+        T, num_heads, dv, L.f32(eps), {"silu": 0, "sigmoid": 1}[gate_kind], int(bool(gate_first)), L.stream_handle()))
     return y
 
 
@@ -81,17 +84,18 @@ def xielu(z: torch.Tensor, params: torch.Tensor, out_dtype: torch.dtype) -> torc
 
 
 def layer_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype,
-               rows: torch.Tensor | None = None) -> torch.Tensor:
-    """y = (x - mean) / sqrt(var + eps) * weight per row (var: the mean of the squared deviations),
-    in 32-bit, written as ``out_dtype``.  ``rows`` (int32) gathers input rows."""
+               rows: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> torch.Tensor:
+    """y = (x - mean) / sqrt(var + eps) * weight (+ bias) per row (var: the mean of the squared
+    deviations), in 32-bit, written as ``out_dtype``.  ``rows`` (int32) gathers input rows."""
     _rows2d(x, "layer_norm")
-    assert weight.dtype == torch.float32 and weight.is_contiguous() and weight.shape == (x.shape[1],)
+    for v in (weight, bias):
+        assert v is None or (v.dtype == torch.float32 and v.is_contiguous() and v.shape == (x.shape[1],))
     if rows is not None:
         assert rows.dtype == torch.int32 and rows.is_contiguous()
     n = x.shape[0] if rows is None else rows.shape[0]
     y = torch.empty((n, x.shape[1]), dtype=out_dtype, device=x.device)
-    L.check(L.core().dsp_layer_norm(L.ptr(x), L.dtype_code(x.dtype), L.i64(x.stride(0)), L.ptr(weight), L.f32(eps),
-                                    L.ptr(rows), L.ptr(y), L.dtype_code(out_dtype), L.i64(y.stride(0)), n, x.shape[1],
+    L.check(L.core().dsp_layer_norm(L.ptr(x), L.dtype_code(x.dtype), L.i64(x.stride(0)), L.ptr(weight), L.ptr(bias),
+                                    L.f32(eps), L.ptr(rows), L.ptr(y), L.dtype_code(out_dtype), L.i64(y.stride(0)), n, x.shape[1],
                                     L.stream_handle()))
     return y
 
@@ -99,12 +103,13 @@ def layer_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: tor
 def stream_update(x32: torch.Tensor, y: torch.Tensor | None, *, gate: torch.Tensor | None = None,
                   scale: torch.Tensor | None = None, rms_weight: torch.Tensor | None = None, rms_eps: float = 0.0,
                   bias: torch.Tensor | None = None, norm_weight: torch.Tensor | None = None, norm_eps: float = 0.0,
-                  norm_kind: str = "layer", out_dtype: torch.dtype | None = None) -> torch.Tensor | None:
+                  norm_kind: str = "layer", norm_bias: torch.Tensor | None = None, y_scale: float = 1.0,
+                  out_dtype: torch.dtype | None = None) -> torch.Tensor | None:
     """x32 += d in place (float32 rows), with d = y * scale * sigmoid(gate) when ``gate`` is given,
-    d = y / sqrt(mean(y^2) + rms_eps) * rms_weight when ``rms_weight`` is, else d = y (``y`` None:
+    d = y / sqrt(mean(y^2) + rms_eps) * rms_weight when ``rms_weight`` is, else d = y * y_scale (``y`` None:
     0); ``bias`` (float32 [width]) is added to every row as well.  With ``out_dtype``: also returns
     the norm of the new rows times ``norm_weight`` (``norm_kind`` "layer": mean taken off; "rms":
-    x / sqrt(mean(x^2) + norm_eps)) or, without ``norm_weight``, the new rows themselves, in that type."""
+    x / sqrt(mean(x^2) + norm_eps)), plus ``norm_bias`` when it is given, or, without ``norm_weight``, the new rows themselves, in that type."""
     _rows2d(x32, "stream_update")
     assert x32.dtype == torch.float32
     if y is not None:
@@ -112,7 +117,8 @@ def stream_update(x32: torch.Tensor, y: torch.Tensor | None, *, gate: torch.Tens
         assert y.shape == x32.shape
     assert norm_kind in ("layer", "rms")
     width = x32.shape[1]
-    for v in (scale, rms_weight, norm_weight, bias):
+    assert y_scale == 1.0 or (gate is None and rms_weight is None)
+    for v in (scale, rms_weight, norm_weight, norm_bias, bias):
         assert v is None or (v.dtype == torch.float32 and v.is_contiguous() and v.shape == (width,))
     if gate is not None:
         _rows2d(gate, "stream_update")
@@ -122,7 +128,8 @@ def stream_update(x32: torch.Tensor, y: torch.Tensor | None, *, gate: torch.Tens
         L.ptr(x32), L.i64(x32.stride(0)), L.ptr(y), L.dtype_code(y.dtype) if y is not None else 0,
         L.i64(y.stride(0) if y is not None else 0), L.ptr(gate),
         L.dtype_code(gate.dtype) if gate is not None else 0, L.i64(gate.stride(0) if gate is not None else 0),
-        L.ptr(scale), L.ptr(rms_weight), L.f32(rms_eps), L.ptr(bias), L.ptr(norm_weight), L.f32(norm_eps),
+        L.ptr(scale), L.ptr(rms_weight), L.f32(rms_eps), L.ptr(bias), L.f32(y_scale), L.ptr(norm_weight),
+        L.ptr(norm_bias), L.f32(norm_eps),
         int(norm_kind == "rms"), L.ptr(out),
         L.dtype_code(out_dtype) if out is not None else 0, L.i64(out.stride(0) if out is not None else 0),
         x32.shape[0], width, L.stream_handle()))

@@ -1,7 +1,8 @@
 """Grouped-query attention over the paged cache: ``gqa_attention`` (keys and values of one
 width, plain softmax) and ``sink_attention`` (widths of their own, a window or a chunked mask,
 an optional sink in the softmax, optional norms of the heads, values optionally blended with
-another layer's or turned by their positions; at the end of this file).
+another layer's or turned by their positions), ``differential_attention`` (two softmax maps per
+head) and ``conv_attention`` (a short convolution on the projections, a window with kept first keys).
 
 q, k, v = h W^T + b (one fused product, rows ordered q, k, v: puneethgv/DiSpec
 dispec/engine/model_runner.py:104-118,131-136); rotation of q and k and the write of k, v
@@ -19,8 +20,9 @@ import torch
 from dispec_b200 import ops
 from dispec_b200.ops import attention as attn_ops
 from dispec_b200.ops import norm32 as norm32_ops
+from dispec_b200.ops import short_conv as conv_ops
 from dispec_b200.cache.manager import CacheTensor
-from dispec_b200.parts.base import CacheNeed, Mixer, TensorSpec
+from dispec_b200.parts.base import CacheNeed, JoinableMixer, Mixer, StateNeed, TensorSpec
 from dispec_b200.registry import register_part
 
 
@@ -322,3 +324,77 @@ class DifferentialAttention(Mixer):
         heads = norm32_ops.diff_heads(maps, H, self.lam, 1.0 - self.diff, self.norm_eps, ctx.dtype,
                                       gate=z[:, n_qkv:] if self.head_gate else None)
         return ops.linear(heads, self.w_o, out_dtype=torch.float32)
+
+
+@register_part("mixer", "conv_attention")
+class ConvAttention(JoinableMixer):
+    """Grouped-query attention with a short convolution on its projections and norms after the rotation:
+
+        q, k, v = C(W_q h + b_q), C(W_k h + b_k), C(W_v h + b_v)     (biases with ``bias``)
+        C: a causal convolution over time per channel, ``taps`` weights a channel (``<name>.conv`` [channels,
+        taps], last column: the current token; zeros before the sequence's start; ``taps`` 0: none)
+        q, k turned by the position encoding (either layout), then, with ``head_norm``, every head divided by
+        its root mean square (``norm_eps`` inside the root, no weight)
+        plain softmax of (q . k_j) * scale over the keys j <= p with p - window < j or j < ``keep_first``
+        (window 0: every j <= p); output W_o on the concatenated heads.
+
+    The last taps - 1 projected rows of a request are its state; keys and values are cached behind
+    convolution, rotation and norm.  Everything between the projections' 32-bit rows and the cache is
+    32-bit, as are scores and softmax.  ``out_scale`` multiplies the values before they are cached."""
+
+    def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int, scale: float,
+                 position_encoding, window: int = 0, keep_first: int = 0, taps: int = 0, bias: bool = True,
+                 head_norm: bool = True, norm_eps: float = 0.0):
+        if num_heads % num_kv_heads:
+            raise ValueError(f"num_heads={num_heads} is not a multiple of num_kv_heads={num_kv_heads}")
+        if not float(scale) > 0.0:
+            raise ValueError(f"the attention scale must be positive, got {scale}")
+        if min(window, keep_first, taps) < 0:
+            raise ValueError(f"conv_attention: window={window}, keep_first={keep_first}, taps={taps} must not be negative")
+        self.hidden_size, self.num_heads, self.num_kv_heads = hidden_size, num_heads, num_kv_heads
+        self.key_dim, self.value_dim, self.scale = key_dim, value_dim, float(scale)
+        self.window, self.keep_first = int(window), int(keep_first) if window else 0
+        self.taps, self.bias, self.head_norm, self.norm_eps = int(taps), bool(bias), bool(head_norm), float(norm_eps)
+        self.position_encoding = position_encoding
+        self.widths = (num_heads * key_dim, num_kv_heads * key_dim, num_kv_heads * value_dim)
+        self.out_columns = num_heads * value_dim
+        self.w_conv = None
+
+    def tensor_specs(self):
+        specs = {"o.weight": TensorSpec((self.hidden_size, self.out_columns))}
+        for name, n in zip("qkv", self.widths):
+            specs[name + ".weight"] = TensorSpec((n, self.hidden_size))
+            if self.bias:
+                specs[name + ".bias"] = TensorSpec((n,))
+            if self.taps:
+                specs[name + ".conv"] = TensorSpec((n, self.taps), dtype="float32", init="one_plus_normal")
+        return specs
+
+    def load(self, tensors):
+        self.w_in = torch.cat([tensors[n + ".weight"] for n in "qkv"], dim=0).contiguous()
+        self.b_in = torch.cat([tensors[n + ".bias"] for n in "qkv"]).contiguous() if self.bias else None
+        self.w_o = tensors["o.weight"]
+        if self.taps:  # [taps, channels]: neighbouring channels side by side
+            self.w_conv = torch.cat([tensors[n + ".conv"] for n in "qkv"], dim=0).t().contiguous()
+
+    def cache_need(self):
+        return CacheNeed((CacheTensor("key", self.num_kv_heads, self.key_dim),
+                          CacheTensor("value", self.num_kv_heads, self.value_dim)), self.window, self.keep_first)
+
+    def state_need(self):
+        return StateNeed((self.taps - 1, sum(self.widths)), "float32") if self.taps > 1 else None
+
+    def tokens_per_attention_tile(self):
+        return attn_ops.sink_tokens_per_tile(self.num_heads // self.num_kv_heads, self.key_dim, self.value_dim)
+
+    def heads(self, ctx, z, cache, state, out):
+        H, G, dk, dv = self.num_heads, self.num_kv_heads, self.key_dim, self.value_dim
+        rot = self.position_encoding.rotation()
+        if rot is not None and rot.magnitude != 1.0:
+            raise ValueError("conv_attention applies pure rotations only (the encoding has a magnitude)")
+        inv_freq, rotary_dim = (rot.inv_freq, rot.rotary_dim) if rot is not None else (None, 0)
+        q = conv_ops.qkv_conv_rotate_store(z, self.w_conv, state.buffer if state is not None else None, ctx, cache, inv_freq,
+                                           rotary_dim, rot is not None and rot.layout == "interleaved", H, G, dk, dv,
+                                           ctx.dtype, self.head_norm, self.norm_eps, self.out_scale)
+        attn_ops.sink_paged_attention(ctx, q, cache, out, H, G, dk, dv, self.window,
+                                      self.scale * self.position_encoding.score_scale(), False, keep_first=self.keep_first)

@@ -15,7 +15,8 @@ Roles and their required methods:
   ``PositionEncoding.score_scale() -> float``: what the attention mixer asks of it.
 * ``Mixer.forward(ctx, x, cache, state) -> y``; ``cache_need()`` says which named tensors
   a call of this mixer keeps per token in the paged cache (or None), ``state_need()`` what
-  fixed-size per-request state (or None).
+  fixed-size per-request state (a need, a tuple of them, or None; ``state`` is then a view, a tuple of
+  views, or None).
 * ``FeedForward.forward(ctx, x) -> y``.
 * ``Block.forward(ctx, x, cache, state) -> x``: the arrangement of two norms, a mixer
   and a feed-forward with their residual sums.
@@ -27,6 +28,7 @@ from typing import Any
 
 import torch
 
+from dispec_b200 import ops
 from dispec_b200.cache.manager import CacheTensor, key_value_tensors  # noqa: F401  (CacheTensor re-exported)
 
 
@@ -61,9 +63,11 @@ class CacheNeed:
     attention keeps two of equal shape, "key" and "value" (``CacheNeed.key_value``); a mixer
     that caches one latent tensor, or keys and values of different widths, lists those instead
     and finds them by name in ``LayerCacheView.tensors``.  ``window`` 0: every token stays;
-    W > 0: only the last W positions are ever read, older pages can be given back."""
+    W > 0: only the last W positions are ever read (and the ``keep_first`` first ones), other pages
+    can be given back."""
     tensors: tuple
     window: int = 0
+    keep_first: int = 0
 
     @classmethod
     def key_value(cls, num_kv_heads: int, head_dim: int, window: int = 0) -> "CacheNeed":
@@ -148,7 +152,7 @@ class Mixer(Part):
     def cache_need(self) -> CacheNeed | None:
         return None
 
-    def state_need(self) -> StateNeed | None:
+    def state_need(self) -> StateNeed | tuple | None:
         return None
 
     def tokens_per_attention_tile(self):
@@ -158,6 +162,29 @@ class Mixer(Part):
 
     def forward(self, ctx, x, cache, state):
         raise NotImplementedError
+
+
+class JoinableMixer(Mixer):
+    """A mixer of the form W_o f(W_in h + b_in): one product into its rows, something of its own on
+    those rows (``heads``), one product out of them.  Another mixer can run several of these side by
+    side as one: their input matrices stacked, each one's ``heads`` on its columns, their output
+    matrices joined along the input dimension (the sum over the mixers is then part of that product).
+
+    ``load`` sets ``w_in`` [columns, hidden], ``b_in`` (or None) and ``w_o`` [hidden, out_columns].
+    ``out_scale``: a factor on the mixer's result, set before ``load``; ``heads`` applies it in 32-bit."""
+    out_scale = 1.0
+    out_columns = 0
+    w_in = b_in = w_o = None
+
+    def heads(self, ctx, z, cache, state, out):
+        """From the rows ``z`` [T, columns] of the input product (float32) to ``out`` [T, out_columns]."""
+        raise NotImplementedError
+
+    def forward(self, ctx, x, cache, state):
+        z = ops.linear(x, self.w_in, self.b_in, out_dtype=torch.float32)
+        out = torch.empty((x.shape[0], self.out_columns), dtype=x.dtype, device=x.device)
+        self.heads(ctx, z, cache, state, out)
+        return ops.linear(out, self.w_o, out_dtype=torch.float32)
 
 
 class FeedForward(Part):

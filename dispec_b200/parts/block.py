@@ -8,6 +8,8 @@ feed-forward output on as ``pending`` so that the next block's first norm (or th
 adds it."""
 from __future__ import annotations
 
+from typing import NamedTuple
+
 import torch
 
 from dispec_b200.ops.gemm import NormedRows
@@ -274,6 +276,53 @@ class OutputNormBlock(Block):
         nxt = norm32_ops.stream_update(full, y, rms_weight=norm.weight, rms_eps=norm.eps,
                                        out_dtype=ctx.dtype if (copies and then_norm is not None) else None)
         return x, nxt
+
+
+class LayerNormTail(NamedTuple):
+    """A layer norm offered to the kernel that writes the rows it reads."""
+    weight: torch.Tensor
+    eps: float
+    bias: torch.Tensor | None
+
+
+@register_part("block", "scaled_pre_norm")
+class ScaledPreNormBlock(Block):
+    """Pre-norm sublayers whose results are multiplied by one number m before the sum, on a residual
+    stream kept in 32-bit floats (``WideStream``):
+
+        x <- x + m mixer(norm1(x));   x <- x + m ffn(norm2(x))            (if there is a feed-forward)
+
+    The norms are layer norms given as parts (``layer_norm_f32``); the sublayers return 32-bit rows.
+    Every sum runs as one kernel with the norm that reads the new stream; the block hands the next
+    block's first norm of its result on as ``pending`` when that block is of this kind too."""
+
+    def __init__(self, hidden_size: int, multiplier: float, mixer_norm, mixer, ffn_norm=None, feed_forward=None):
+        if (ffn_norm is None) != (feed_forward is None):
+            raise ValueError("scaled_pre_norm: a feed-forward and its norm come together or not at all")
+        self.hidden_size, self.multiplier = hidden_size, float(multiplier)
+        self.mixer_norm, self.mixer = mixer_norm, mixer
+        self.ffn_norm, self.feed_forward = ffn_norm, feed_forward
+
+    def first_norm_after_product(self):
+        return LayerNormTail(self.mixer_norm.weight, self.mixer_norm.eps, self.mixer_norm.bias)
+
+    def _sum(self, ctx, full, y, tail):
+        if tail is None:
+            return norm32_ops.stream_update(full, y, y_scale=self.multiplier)
+        return norm32_ops.stream_update(full, y, y_scale=self.multiplier, norm_weight=tail.weight, norm_eps=tail.eps,
+                                        norm_bias=tail.bias, out_dtype=ctx.dtype)
+
+    def forward(self, ctx, x, pending, cache, state, then_norm=None):
+        if not isinstance(x, WideStream) or x.full.dtype != torch.float32:
+            raise ValueError("scaled_pre_norm: the residual stream must be a 32-bit WideStream")
+        if then_norm is not None and not isinstance(then_norm, LayerNormTail):
+            raise ValueError("scaled_pre_norm: the block after this one takes its first norm in another form")
+        h = pending if pending is not None else self.mixer_norm.forward(ctx, x)
+        y = self.mixer.forward(ctx, h, cache, state)
+        if self.feed_forward is not None:
+            h = self._sum(ctx, x.full, y, LayerNormTail(self.ffn_norm.weight, self.ffn_norm.eps, self.ffn_norm.bias))
+            y = self.feed_forward.forward(ctx, h)
+        return x, self._sum(ctx, x.full, y, then_norm)
 
 
 @register_part("stream_input", "pass_entry")

@@ -15,6 +15,10 @@ with one gain of size vdim shared by the heads, then projected.
 no other scale; the concatenated heads are RMS-normed together with one gain over all of them,
 multiplied by sigmoid(W_g h) and projected.
 
+``gated_linear_attention``: a decay per key channel and token, a_t = sigmoid(z)^(1/tau) with
+z = W_a2 (W_a1 h) + bias, q scaled by dim^(-1/2), b_t = k_t; every head's o is RMS-normed with one gain of
+size vdim, multiplied by silu(W_g h) and projected.
+
 All run one fused projection, the recurrence kernel (which forms a_t, b_t, q_t from the raw
 projection rows in 32-bit), the per-head norm kernel and the output projection.
 """
@@ -136,4 +140,38 @@ class Lightning(_MatrixStateMixer):
             ctx.positions, decay=self.decay, silu_inputs=True)
         gated = norm32_ops.head_norm_gate(o, 1, self.eps, x.dtype, gain=self.gain,
                                           gate=proj[:, 2 * H * d + H * dv:], gate_kind="sigmoid")
+        return ops.linear(gated, self.w_o, out_dtype=torch.float32)
+
+
+@register_part("mixer", "gated_linear_attention")
+class GatedLinearAttention(_MatrixStateMixer):
+    def __init__(self, hidden_size: int, num_heads: int, dim: int, vdim: int, rank: int, tau: float, eps: float):
+        super().__init__(hidden_size, num_heads, dim, vdim, eps)
+        if rank <= 0 or not float(tau) > 0.0:
+            raise ValueError(f"gated_linear_attention: rank={rank} and tau={tau} must be positive")
+        self.rank, self.tau = int(rank), float(tau)
+        self.gate_map = self.gate_bias = self.gain = None
+
+    def tensor_specs(self):
+        h, H, d, dv, r = self.hidden_size, self.num_heads, self.dim, self.vdim, self.rank
+        return {"q.weight": TensorSpec((H * d, h)), "k.weight": TensorSpec((H * d, h)), "v.weight": TensorSpec((H * dv, h)),
+                "g.weight": TensorSpec((H * dv, h)), "o.weight": TensorSpec((h, H * dv)),
+                "a1.weight": TensorSpec((r, h)), "a2.weight": TensorSpec((H * d, r), dtype="float32"),
+                "a2.bias": TensorSpec((H * d,), dtype="float32", init="zeros"),
+                "norm.weight": TensorSpec((dv,), dtype="float32", init="one_plus_normal")}
+
+    def load(self, tensors):
+        self.w_in = torch.cat([tensors[n + ".weight"] for n in ("q", "k", "v", "g", "a1")], dim=0).contiguous()
+        self.gate_map = tensors["a2.weight"].t().contiguous()  # [rank, H * dim]
+        self.gate_bias, self.gain, self.w_o = tensors["a2.bias"], tensors["norm.weight"], tensors["o.weight"]
+
+    def forward(self, ctx, x, cache, state):
+        H, d, dv = self.num_heads, self.dim, self.vdim
+        proj = ops.linear(x, self.w_in, out_dtype=torch.float32)  # [T, q | k | v | g | a1]
+        v_off, g_off = 2 * H * d, 2 * H * d + H * dv
+        o = rec_ops.linear_recurrence(
+            proj, 0, H * d, v_off, rec_ops.KEY_DECAY, H, d, dv, state.buffer, state.slots, ctx.q_start, ctx.positions,
+            gate_map=self.gate_map, gate_bias=self.gate_bias, low_off=g_off + H * dv, q_scale=d ** -0.5,
+            power=1.0 / self.tau)
+        gated = norm32_ops.head_norm_gate(o, H, self.eps, x.dtype, gain=self.gain, gate=proj[:, g_off:g_off + H * dv])
         return ops.linear(gated, self.w_o, out_dtype=torch.float32)

@@ -64,7 +64,8 @@ class GatedMoE(FeedForward):
         g = min(W_gate_e a, limit),  u = clamp(W_up_e a, -limit, limit).
 
     Router logits z = W_router h in 32-bit (the router matrix stays float32 in every mode);
-    scores s = sigmoid(z) (``score`` "sigmoid") or softmax(z); groups of experts as in
+    scores s = sigmoid(z) (``score`` "sigmoid") or softmax(z), or the logits themselves, turned into
+    weights by a softmax over the chosen ones ("chosen_softmax"); groups of experts as in
     ``grouped_moe``; the ``top`` largest scores name the token's experts and are their weights w,
     not renormalised.  ``weight_on`` "input": the output is the sum of expert_e(w h) (the factor is
     applied to the 32-bit sums W_gate_e h and W_up_e h, which is the same product, before the
@@ -75,14 +76,15 @@ class GatedMoE(FeedForward):
     (u + up_shift) (no limit, alpha 1 and up_shift 0: silu(W_gate a) * (W_up a)).  ``group_score``
     "top2_sum": a group's score is the sum of its two largest scores (default: its largest).
     ``normalize``: the weights are the chosen scores divided by their sum (+ 1e-20), times
-    ``weight_scale``.  ``shared_gate``: the shared part's result is multiplied by sigmoid(w_sg . h),
+    ``weight_scale``.  ``router_bias``: z = W_router h + ``router.bias`` (float32).
+    ``shared_gate``: the shared part's result is multiplied by sigmoid(w_sg . h),
     one number per token (tensor ``shared_gate.weight`` [1, hidden_size], float32: its row rides in
     the router's product)."""
 
     def __init__(self, hidden_size: int, intermediate_size: int, num_experts: int, top: int, limit: float | None,
                  alpha: float = 1.702, score: str = "sigmoid", weight_on: str = "input", num_groups: int = 1,
                  keep_groups: int = 1, shared=None, up_shift: float = 1.0, group_score: str = "max",
-                 normalize: bool = False, weight_scale: float = 1.0, shared_gate: bool = False):
+                 normalize: bool = False, weight_scale: float = 1.0, shared_gate: bool = False, router_bias: bool = False):
         if num_experts <= 0 or num_groups <= 0 or num_experts % num_groups:
             raise ValueError(f"glu_moe: {num_experts} experts do not form {num_groups} equal groups")
         if not 0 < keep_groups <= num_groups:
@@ -90,7 +92,7 @@ class GatedMoE(FeedForward):
         if not 0 < top <= keep_groups * (num_experts // num_groups):
             raise ValueError(f"glu_moe: top={top} experts cannot come from {keep_groups} groups of "
                              f"{num_experts // num_groups}")
-        if score not in ("sigmoid", "softmax") or weight_on not in ("input", "output"):
+        if score not in ("sigmoid", "softmax", "chosen_softmax") or weight_on not in ("input", "output"):
             raise ValueError(f"glu_moe: score={score!r} / weight_on={weight_on!r} are not known")
         limit = float("inf") if limit is None else limit
         if not limit > 0:
@@ -99,6 +101,7 @@ class GatedMoE(FeedForward):
             raise ValueError(f"glu_moe: group_score={group_score!r} is not known")
         if shared_gate and shared is None:
             raise ValueError("glu_moe: a gate on the shared part but no shared part")
+        self.router_bias, self.b_router = bool(router_bias), None
         self.up_shift, self.group_score = float(up_shift), group_score
         self.normalize, self.weight_scale, self.shared_gate = bool(normalize), float(weight_scale), bool(shared_gate)
         self.hidden_size, self.intermediate_size = hidden_size, intermediate_size
@@ -115,6 +118,8 @@ class GatedMoE(FeedForward):
             specs[f"experts.{e}.down.weight"] = TensorSpec((h, i))
         if self.shared_gate:
             specs["shared_gate.weight"] = TensorSpec((1, h), dtype="float32")
+        if self.router_bias:
+            specs["router.bias"] = TensorSpec((self.num_experts,), dtype="float32")
         return specs
 
     def load(self, tensors):
@@ -122,6 +127,9 @@ class GatedMoE(FeedForward):
         self.w_router = tensors["router.weight"]
         if self.shared_gate:
             self.w_router = torch.cat([self.w_router, tensors["shared_gate.weight"]], dim=0).contiguous()
+        if self.router_bias:
+            self.b_router = torch.cat([tensors["router.bias"], torch.zeros_like(tensors["router.bias"][:1])]).contiguous() \
+                if self.shared_gate else tensors["router.bias"]
         # rows of the gate and up matrices in turn: the product's epilogue holds a gate and its up
         # value in one thread and writes the unit's result
         self.w_gate_up = torch.stack(
@@ -132,7 +140,7 @@ class GatedMoE(FeedForward):
     def forward(self, ctx, x):
         routed = moe_ops.route(x, self.w_router, self.num_groups, self.keep_groups, self.top, score=self.score,
                                group_score=self.group_score, normalize=self.normalize, weight_scale=self.weight_scale,
-                               extra_rows=1 if self.shared_gate else 0)
+                               extra_rows=1 if self.shared_gate else 0, bias=self.b_router)
         ids, wts = routed[0], routed[1]
         plan = moe_ops.plan(ids, self.num_experts, moe_ops.tensor_cores_supported(x.dtype, self.hidden_size,
                                                                                    self.intermediate_size))

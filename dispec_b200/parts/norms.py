@@ -99,21 +99,25 @@ class ScalarRMSNorm32(RMSNorm32):
 
 @register_part("norm", "layer_norm_f32")
 class LayerNorm32(Norm):
-    """y = (x - mean) / sqrt(var + eps) * w with a gain and no bias (var: the mean of the squared
-    deviations), everything in 32-bit; the gain is float32 in every mode.  Reads a 32-bit stream
-    (``WideStream``) or a plain tensor; the result comes in ``ctx.dtype`` (what a product reads)."""
+    """y = (x - mean) / sqrt(var + eps) * w with a gain and, with ``with_bias``, + b (var: the mean of
+    the squared deviations), everything in 32-bit; gain and bias are float32 in every mode.  Reads a
+    32-bit stream (``WideStream``) or a plain tensor; the result comes in ``ctx.dtype`` (what a product reads)."""
 
-    def __init__(self, hidden_size: int, eps: float):
+    def __init__(self, hidden_size: int, eps: float, with_bias: bool = False):
         self.hidden_size = hidden_size
         self.eps = float(eps)
-        self.weight = None
+        self.with_bias = bool(with_bias)
+        self.weight = self.bias = None
 
     def tensor_specs(self):
-        return {"weight": TensorSpec((self.hidden_size,), dtype="float32", init="one_plus_normal")}
+        specs = {"weight": TensorSpec((self.hidden_size,), dtype="float32", init="one_plus_normal")}
+        if self.with_bias:
+            specs["bias"] = TensorSpec((self.hidden_size,), dtype="float32")
+        return specs
 
     def load(self, tensors):
-        self.weight = tensors["weight"]
+        self.weight, self.bias = tensors["weight"], tensors.get("bias")
 
     def forward(self, ctx, x, rows=None):
         full = x.full if isinstance(x, WideStream) else x
-        return norm32_ops.layer_norm(full, self.weight, self.eps, ctx.dtype, rows=rows)
+        return norm32_ops.layer_norm(full, self.weight, self.eps, ctx.dtype, rows=rows, bias=self.bias)

@@ -14,7 +14,12 @@ hi = min(ceil(n(slow)), rotary_dim - 1) and ramp_i = clamp((i - lo) / max(hi - l
 pair i turns at inv_freq[i] / factor * ramp_i + inv_freq[i] * (1 - ramp_i): fast pairs keep their
 frequency, slow pairs are divided by ``factor``, those between are blended.  Cosine and sine are
 then multiplied by 0.1 ln(factor) + 1 (``Rotation.magnitude``), which a mixer's kernels apply to
-queries and keys alike."""
+queries and keys alike.
+
+``banded`` = (factor, low, high, original): another slowing by wavelength l = 2 pi / inv_freq, with no
+magnitude: pairs with l < original / high keep their frequency, pairs with l > original / low are
+divided by ``factor``, and between the two s = (original / l - low) / (high - low) blends
+(1 - s) inv_freq / factor + s inv_freq."""
 from __future__ import annotations
 
 import math
@@ -28,7 +33,7 @@ from dispec_b200.registry import register_part
 @register_part("position_encoding", "rotary")
 class RotaryEncoding(PositionEncoding):
     def __init__(self, head_dim: int, theta: float, rotary_dim: int | None = None, layout: str = "halves",
-                 exact_table: bool = False, slowed: tuple | None = None):
+                 exact_table: bool = False, slowed: tuple | None = None, banded: tuple | None = None):
         if layout not in ("halves", "interleaved"):
             raise ValueError(f"rotary layout {layout!r} is not one of 'halves', 'interleaved'")
         self.layout = layout
@@ -50,9 +55,18 @@ class RotaryEncoding(PositionEncoding):
                                  f"theta={self.theta} do not describe one")
             self.slowed = (factor, original, fast, slow)
             self.magnitude = 0.1 * math.log(factor) + 1.0
+        self.banded = None
+        if banded is not None:
+            if slowed is not None:
+                raise ValueError("a rotation is slowed in one way or the other, not in both")
+            factor, low, high, original = (float(v) for v in banded)
+            if not (factor > 0.0 and original > 0.0 and 0.0 < low <= high):
+                raise ValueError(f"banded rotation: factor={factor} low={low} high={high} original={original} "
+                                 f"do not describe one")
+            self.banded = (factor, low, high, original)
 
     def prepare(self, device):
-        wide = torch.float64 if (self.exact_table or self.slowed) else torch.float32
+        wide = torch.float64 if (self.exact_table or self.slowed or self.banded) else torch.float32
         exponent = torch.arange(0, self.rotary_dim, 2, dtype=wide) / self.rotary_dim
         freq = 1.0 / (self.theta ** exponent)
         if self.slowed is not None:
@@ -62,6 +76,12 @@ class RotaryEncoding(PositionEncoding):
             hi = min(math.ceil(turns(slow)), self.rotary_dim - 1)
             ramp = ((torch.arange(self.rotary_dim // 2, dtype=wide) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
             freq = freq / factor * ramp + freq * (1.0 - ramp)
+        if self.banded is not None:
+            factor, low, high, original = self.banded
+            turns = original * freq / (2 * math.pi)  # original / wavelength
+            s = (turns - low) / (high - low) if high > low else torch.ones_like(turns)
+            blend = (1.0 - s) * freq / factor + s * freq
+            freq = torch.where(turns > high, freq, torch.where(turns < low, freq / factor, blend))
         self.inv_freq = freq.to(torch.float32).to(device)
 
     def rotation(self):

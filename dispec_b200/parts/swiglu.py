@@ -1,5 +1,6 @@
-"""Dense SwiGLU feed-forward: down( silu(h Wg^T) * (h Wu^T) ), gate and up as one fused
-product (puneethgv/DiSpec dispec/engine/model_runner.py:112,222-226), no biases."""
+"""Dense gated feed-forward: down( act(h Wg^T) * (h Wu^T) ), gate and up as one fused product,
+no biases; ``act`` is silu (puneethgv/DiSpec dispec/engine/model_runner.py:112,222-226) or the
+tanh form of gelu."""
 from __future__ import annotations
 
 import torch
@@ -12,7 +13,10 @@ from dispec_b200.registry import register_part
 
 @register_part("feed_forward", "swiglu")
 class SwiGLUFeedForward(FeedForward):
-    def __init__(self, hidden_size: int, intermediate_size: int, out_float32: bool = False):
+    def __init__(self, hidden_size: int, intermediate_size: int, out_float32: bool = False, act: str = "silu"):
+        if act not in ops.GLU_ACTS:
+            raise ValueError(f"swiglu: activation {act!r} is not one of {', '.join(ops.GLU_ACTS)}")
+        self.act = act
         self.hidden_size = hidden_size
         self.intermediate_size = intermediate_size
         # True: the down product returns 32-bit rows (for an arrangement that norms or sums them in 32-bit)
@@ -46,9 +50,9 @@ class SwiGLUFeedForward(FeedForward):
         comes back.  ``x`` may be a norm still to be applied (``NormedRows``), and ``then_norm``
         the (weight, eps) of the norm that reads the result: then (result, NormedRows) comes back."""
         if self.block and gemm_ops.gate_up_swiglu_supported(x, self.w_gate_up):
-            act = gemm_ops.linear_gate_up_swiglu(x, self.w_gate_up)
+            act = gemm_ops.linear_gate_up_swiglu(x, self.w_gate_up, act=self.act)
         else:
-            act = ops.swiglu(ops.linear(x, self.w_gate_up), block=self.block)
+            act = ops.swiglu(ops.linear(x, self.w_gate_up), block=self.block, act=self.act)
         if self.out_float32:
             if residual is not None or then_norm is not None:
                 raise ValueError("swiglu: 32-bit rows go to an arrangement that does the sum itself")

@@ -105,6 +105,7 @@ def load_model(folder: str, dtype="bfloat16", device="cuda:0") -> DecoderModel:
     """A model folder (config.json + safetensors) -> a model on the device.  Same role and
     argument order as the reference's ``load_model(name, dtype, device)``
     (puneethgv/DiSpec dispec/models/loader.py:18-27)."""
-    config = load_model_config(read_config_json(folder))
+    source = CheckpointFolder(folder)
+    config = load_model_config(read_config_json(folder)).with_tensor_shapes(source)
     model = build_model(config)
-    return load_into(model, CheckpointFolder(folder), dtype, device, where=folder)
+    return load_into(model, source, dtype, device, where=folder)
