@@ -996,6 +996,135 @@ def milivik_points(args, pk: dict) -> dict:
     return out
 
 
+# ------------------------------------------------------------ Bepepel beside Murutar at equal size
+# Bepepel's closest relative in this package is Murutar (linear attention with a matrix state and
+# windowed attention in turn, gated units, experts, layer norms in front of the sublayers of a 32-bit
+# stream).  Both with eight layers at the same width, heads, head sizes, window, vocabulary, number of
+# experts and feed-forward weights a token passes.  Bepepel: gla + dense, parallel + experts, gla +
+# experts twice; that period twice; 16 experts of a quarter of the dense width of which 2 are used
+# and a shared expert of half of it.  The state-space side of a parallel layer is as wide as the model
+# (heads of 64, states of 128 rows).  Murutar: lightning + dense, attention + experts, lightning +
+# experts twice; that period twice; 16 experts of half the dense width of which 2 are used.
+BEPEPEL_LAYERS = 8
+
+
+def bepepel_config(shape: str) -> dict:
+    z = MURUTAR_SHAPES[shape]
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // 4}, "router": {"experts": z["experts"], "top": z["top"]},
+           "shared": {"ff": z["ff"] // 2}}
+    gla = lambda mlp: {"type": "gla", "mlp": mlp, "mixer": {"heads": z["heads"], "dim": z["dim"], "vdim": z["vdim"], "tau": 16.0}}
+    par = {"type": "parallel", "mlp": moe, "mixer": {
+        "left_scale": 1.0, "right_scale": 1.0,
+        "left": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "conv": 4,
+                 "scale": z["dim"] ** -0.5, "mask": {"size": z["window"], "keep_first": 16},
+                 "rot": {"dims": z["rot"], "base": 1e6, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}},
+        "right": {"heads": z["width"] // 64, "vdim": 64, "state": 128, "groups": 2, "conv": 4, "norm_groups": 2}}}
+    return {"architecture": "Bepepel", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "logit_scale": 1.0, "layers": [gla(dense), par, gla(moe), gla(moe)] * (BEPEPEL_LAYERS // 4)}
+
+
+def murutar_mostly_linear_config(shape: str) -> dict:
+    cfg = murutar_config(shape)
+    lin_dense, _, lin_moe, att_moe = cfg["layers"][:4]
+    cfg["layers"] = [lin_dense, att_moe, lin_moe, lin_moe] * (BEPEPEL_LAYERS // 4)
+    return cfg
+
+
+def bepepel_bytes_and_flops(cfg: dict, rank: int = 16):
+    """As ``murutar_bytes_and_flops``; states are read and written once a decode step."""
+    W, V = cfg["width"], cfg["vocab"]
+    fixed, cache_layers, state_bytes, attn, rec, expert_layers = 0, [], 0, [], 0, []
+    for e in cfg["layers"]:
+        m, mlp = e["mixer"], e["mlp"]
+        if e["type"] == "gla":
+            H, d, dv = m["heads"], m["dim"], m["vdim"]
+            n = (2 * H * d + 2 * H * dv + rank) * W + 2 * H * d * rank + W * H * dv
+            state_bytes += 2 * H * d * dv * 4
+            rec += 4 * H * d * dv
+        else:
+            a, s = m["left"], m["right"]
+            H, G, d, dv = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            inner, N = s["heads"] * s["vdim"], s["state"]
+            channels = inner + 2 * s["groups"] * N
+            n = (H * d + G * d + G * dv) * W + W * H * dv + (inner + channels + s["heads"]) * W + W * inner
+            cache_layers.append((G * (d + dv) * 2, a["mask"]["size"] + a["mask"]["keep_first"]))
+            attn.append((H * (d + dv), a["mask"]["size"] + a["mask"]["keep_first"]))
+            state_bytes += 2 * 4 * (s["heads"] * N * s["vdim"] + (s["conv"] - 1) * channels + (a["conv"] - 1) * (H * d + G * (d + dv)))
+            rec += 4 * s["heads"] * N * s["vdim"]
+        if mlp["kind"] == "dense":
+            n += 3 * mlp["ff"] * W
+        else:
+            r = mlp["router"]
+            n += r["experts"] * W * 2 + 3 * mlp["shared"]["ff"] * W  # float32 router
+            expert_layers.append((r["experts"], r["top"], 3 * mlp["expert"]["ff"] * W))
+        fixed += n
+
+    def weight_bytes(batch):
+        return 2 * (fixed + V * W + sum(min(E, batch * top) * w for E, top, w in expert_layers))
+
+    def cache_bytes(ctx):
+        return sum(per * min(ctx, win) for per, win in cache_layers)
+
+    def prefill_flops(T):
+        f = 2 * T * (fixed + sum(top * w for _, top, w in expert_layers)) + rec * T + 2 * V * W
+        for per, win in attn:
+            f += 2 * per * sum(min(t + 1, win) for t in range(T))
+        return f
+
+    total = 2 * (fixed + V * W + sum(E * w for E, _, w in expert_layers))
+    return weight_bytes, cache_bytes, state_bytes, prefill_flops, total
+
+
+def bepepel_points(args, pk: dict) -> dict:
+    """Prefill (2,048 tokens in one step) and decode (batch 1, 8, 64 from captured graphs, 1,536
+    tokens into the sequence) of Bepepel and of Murutar with as many layers, at equal sizes, each
+    with the fraction of its own roofline."""
+    import torch
+    from dispec_b200 import load_model_config
+    from dispec_b200.engine import ModelRunner
+    from dispec_b200.weights import load_random_model
+    prompt_len = PROMPT_LEN + PROMPT_LEN // 2
+    out = {"only": "bepepel", "layers": BEPEPEL_LAYERS, "prompt_len": prompt_len, "prefill_tokens": PREFILL_TOKENS, "peaks": pk}
+    steps, warmup = max(20, min(args.steps, 50)), max(3, args.warmup // 2)
+    per_req = (prompt_len + NEW_TOKENS + steps + warmup + PAGE_SIZE) // PAGE_SIZE + 1
+    shapes = ["1.5b"] if args.no_other_shapes else list(MURUTAR_SHAPES)
+    for shape in shapes:
+        for family in ("bepepel", "murutar"):
+            if family == "bepepel":
+                cfg_dict = bepepel_config(shape)
+                weight_bytes, cache_bytes, state_bytes, prefill_flops, total = bepepel_bytes_and_flops(cfg_dict)
+            else:
+                cfg_dict = murutar_mostly_linear_config(shape)
+                weight_bytes, cache_bytes, state_bytes, prefill_flops, total = murutar_bytes_and_flops(cfg_dict)
+            vocab = cfg_dict["vocab"]
+            model = load_random_model(load_model_config(cfg_dict), 5, STD, "bfloat16", "cuda:0")
+            torch.cuda.synchronize()
+            key = f"{family}_{shape}"
+            out[f"{key}_weight_gb"] = round(total / 1e9, 3)
+            for b in (1, 8, 64):
+                r = ModelRunner(model, page_size=PAGE_SIZE, num_pages=max(b * per_req, 160), max_num_seqs=max(b, 8),
+                                cuda_graph=True)
+                ms, launches, ctx = decode_direct(r, random_prompts(b, prompt_len, vocab, 13 + b), steps, warmup)
+                step_bytes = weight_bytes(b) + b * (cache_bytes(ctx) + state_bytes)
+                out[f"{key}_decode_b{b}"] = round(b * 1000.0 / ms, 1)
+                out[f"{key}_decode_b{b}_ms"] = round(ms, 4)
+                out[f"{key}_decode_b{b}_hbm_frac"] = round(step_bytes / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)
+                out[f"{key}_decode_b{b}_launches_per_step"] = launches // steps
+                print(f"bench: {key} decode at batch {b}: {ms:.3f} ms a step", file=sys.stderr, flush=True)
+                if b == 1:
+                    pms = prefill_time(r, random_prompts(1, PREFILL_TOKENS, vocab, 12)[0], repeats=3)
+                    out[f"{key}_prefill"] = round(PREFILL_TOKENS / pms * 1000.0, 1)
+                    out[f"{key}_prefill_ms"] = round(pms, 3)
+                    out[f"{key}_prefill_frac"] = round(prefill_flops(PREFILL_TOKENS) / (pms * 1e-3) / (pk["bf16_tflops"] * 1e12), 4)
+                del r
+                torch.cuda.empty_cache()
+            del model
+            torch.cuda.empty_cache()
+            print(f"bench: {key} done", file=sys.stderr, flush=True)
+    return out
+
+
 def run_ours(args) -> dict:
     import torch
     from dispec_b200 import load_model_config
@@ -1018,6 +1147,8 @@ def run_ours(args) -> dict:
         return desalix_points(args, peaks())
     if args.only == "milivik":
         return milivik_points(args, peaks())
+    if args.only == "bepepel":
+        return bepepel_points(args, peaks())
     cfg_dict = dict(BENCH_CONFIG)
     seed = SEED
     if args.shape != "1.5b":
@@ -1187,7 +1318,7 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the configuration (recorded)")
     ap.add_argument("--shape", choices=["1.5b", "7b", "14b"], default="1.5b",
                     help="layer sizes: Qwen2.5-1.5B (the default and the recorded configuration), 7B or 14B")
-    ap.add_argument("--only", choices=["decode", "prefill", "timeline", "mma-rate", "tma-rate", "attn-prefill", "puludra", "murutar", "desalix", "milivik"],
+    ap.add_argument("--only", choices=["decode", "prefill", "timeline", "mma-rate", "tma-rate", "attn-prefill", "puludra", "murutar", "desalix", "milivik", "bepepel"],
                     default=None,
                     help="profiling aid: run one phase only and print a short line; timeline: where the time of the "
                          "decode step's products and attention goes (a build with timestamps); mma-rate: cycles per "
@@ -1196,7 +1327,7 @@ def main() -> int:
                          "alone, by shape, length and the order of the pages; puludra: prefill and decode of the Puludra design beside "
                          "Qwen2 at equal width, depth, vocabulary and feed-forward width (eight layers each), with roofline fractions; "
                          "murutar: the same for the Murutar design beside Puludra; desalix: the same for the Desalix design beside "
-                         "Murutar with attention and experts in every layer; milivik: the same for the Milivik design beside Desalix")
+                         "Murutar with attention and experts in every layer; milivik: the same for the Milivik design beside Desalix; bepepel: the same for the Bepepel design beside Murutar")
     ap.add_argument("--batch", type=int, default=BATCH, help="batch of the --only decode phase")
     ap.add_argument("--max-key-ranges", type=int, default=0,
                     help="profiling aid: cap on the key ranges per decoded row beyond one cluster (1: none)")

@@ -21,15 +21,18 @@
 //                 token and head and the value scaled by another (`steps`); o_t gets skip[head] * v_t on top:
 //                     S_t = a S_(t-1) + step b_t v_t^T,   o_t = S_t^T q_t + skip v_t
 //
-// One block per (request, head, tile of value columns).  A thread holds ROWS state rows of one
-// column in registers, four neighbouring rows at a time; the SLICES threads that share a column sit
-// in adjacent lanes and add their partial outputs by shuffles.  Tokens are staged through shared
-// memory in rounds of `tokens_per_round`.  The recurrence is sequential in the tokens of a request,
-// so what can be done ahead of it is: for portions of prompts a first, fully parallel kernel writes
-// q_t, b_t (and a_t) of every token as floats, and the recurrence kernel only streams them in with
-// cp.async, the next round arriving while the current one is computed; single tokens are
-// transformed as they are staged, in one kernel (STEP_DECAY streams the rows themselves always).  A request whose first row carries a negative
-// position (a padding row of a captured step) is skipped: its state slot belongs to someone else.
+// One block of four warps per (request, head, tile of value columns); what a block computes is
+// sequential in the tokens of its request.  A thread holds a tile of the state in registers, four
+// neighbouring rows (twice four beyond 128 rows) of four neighbouring columns, so that what it
+// reads of q, b and a serves four columns and what it reads of v serves four rows.  The SLICES lanes
+// that share columns cover the rows; eight tokens' partial outputs are added over them together, each
+// exchange halving the values a lane still holds, and end up one to a lane.  Tokens are staged through shared
+// memory in rounds: for portions of prompts a first, fully parallel kernel writes q_t, b_t (and a_t) of
+// every token as floats (STEP_DECAY streams its rows as they are), and the recurrence streams them in
+// with cp.async, three rounds ahead of the one that is computed; single tokens are transformed as they
+// are staged, in one kernel.  State rows beyond 256 take a kernel of their own with one column a
+// thread.  A request whose first row carries a negative position (a padding row of a captured step) is
+// skipped: its state slot belongs to someone else.
 #include "common.cuh"
 
 namespace {
@@ -58,6 +61,7 @@ struct RecurrenceArgs {
   const float* steps;      // [T, 2, H]           STEP_DECAY: factor on the value, decay
   const float* skip;       // [H]                 STEP_DECAY
   int heads_per_group;     //                     STEP_DECAY (1 otherwise)
+  int streamed;            // rounds arrive by cp.async ahead of the computation (tile kernel)
   float* state;            // [slots, H, dim, vdim]
   const int* state_slot;   // [S]
   const int* q_start;      // [S + 1]
@@ -178,7 +182,8 @@ __device__ __forceinline__ void cp_async16(float* smem, const float* gmem) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem));
 }
 
-// ROWS: state rows a thread holds; TPR: tokens per staging round; KIND: what a_t is
+// The kernel for more than 256 state rows: a thread holds ROWS rows of one column.  ROWS: state rows a
+// thread holds; TPR: tokens per staging round; KIND: what a_t is
 template <int ROWS, int TPR, int KIND>
 __global__ void __launch_bounds__(THREADS)
 linear_recurrence_kernel(const RecurrenceArgs p) {
@@ -361,6 +366,267 @@ linear_recurrence_kernel(const RecurrenceArgs p) {
   }
 }
 
+// The kernel for up to 256 state rows.  SLICES lanes times QUADS times four rows cover the state's rows.
+constexpr int TILE_WARPS = 4, TILE_THREADS = 32 * TILE_WARPS, TILE_STAGES = 4, BATCH = 8;
+
+template <int SLICES, int QUADS, int KIND>
+struct Tile {
+  static constexpr bool gate = KIND == VECTOR_DECAY, per_token = KIND == TOKEN_DECAY;
+  static constexpr int planes = gate ? 3 : 2;
+  static constexpr int rows = SLICES * 4 * QUADS;                     // state rows, padded
+  static constexpr int cols = TILE_WARPS * (32 / SLICES) * 4;         // value columns of a block
+  static constexpr int round = QUADS == 1 ? 16 : 8;                   // tokens staged together
+  static constexpr int stage = planes * round * rows + round * cols + (per_token ? 2 * round : 0);
+  static constexpr size_t smem(int stages) { return sizeof(float) * stages * stage; }
+};
+
+template <int SLICES, int QUADS, int KIND>
+__global__ void __launch_bounds__(TILE_THREADS)
+recurrence_tile_kernel(const RecurrenceArgs p) {
+  using L = Tile<SLICES, QUADS, KIND>;
+  constexpr bool gate = L::gate, per_token = L::per_token;
+  constexpr int DP = L::rows, C = L::cols, R = L::round, planes = L::planes;
+  extern __shared__ __align__(16) float tile_smem[];
+  const int seq = blockIdx.z, head = blockIdx.y;
+  const int t0 = p.q_start[seq], t1 = p.q_start[seq + 1];
+  if (t1 <= t0 || p.positions[t0] < 0) return;
+  const int tid = threadIdx.x, lane = tid & 31, slice = lane % SLICES;
+  const int cg = (tid >> 5) * (32 / SLICES) + lane / SLICES;  // this thread's group of four columns
+  const int col0 = blockIdx.x * C + cg * 4;
+  const bool streamed = p.streamed != 0;
+  const float* rows = reinterpret_cast<const float*>(p.proj);
+  const bool whole = p.ld % 4 == 0 && (((uintptr_t)rows) & 15) == 0;
+  const bool wide = p.dim % 4 == 0 && (per_token ? whole && p.q_off % 4 == 0 && p.k_off % 4 == 0 : (((uintptr_t)p.ready) & 15) == 0);
+  const bool v_async = p.proj_dtype == DSP_F32;
+  const bool v_wide = whole && p.v_off % 4 == 0 && p.vdim % 4 == 0;
+  const int hd = p.H * p.dim, group0 = (head / p.heads_per_group) * p.dim;
+
+  // state rows q * SLICES * 4 + slice * 4 + e (e < 4) of columns col0 .. col0 + 3
+  float* sp = p.state + (((size_t)p.state_slot[seq] * p.H + head) * p.dim) * p.vdim;
+  const bool s_wide = p.vdim % 4 == 0;
+  float S[QUADS * 4][4];
+#pragma unroll
+  for (int k = 0; k < QUADS * 4; ++k) {
+    const int i = (k >> 2) * (SLICES * 4) + slice * 4 + (k & 3);
+    S[k][0] = S[k][1] = S[k][2] = S[k][3] = 0.f;
+    if (i >= p.dim || col0 >= p.vdim) continue;
+    const float* src = sp + (size_t)i * p.vdim + col0;
+    if (s_wide) {
+      const float4 v = *reinterpret_cast<const float4*>(src);
+      S[k][0] = v.x, S[k][1] = v.y, S[k][2] = v.z, S[k][3] = v.w;
+    } else {
+#pragma unroll
+      for (int c = 0; c < 4; ++c)
+        if (col0 + c < p.vdim) S[k][c] = src[c];
+    }
+  }
+  const float decay = KIND == SCALAR_DECAY ? p.decay[head] : 0.f;
+  const float skip = per_token ? p.skip[head] : 0.f;
+
+  // rows and columns beyond the head's own stay zero in every stage: written here and never again
+  if (DP > p.dim || (int)(blockIdx.x + 1) * C > p.vdim) {
+    for (int idx = tid; idx < (streamed ? TILE_STAGES : 1) * L::stage; idx += TILE_THREADS) tile_smem[idx] = 0.f;
+    __syncthreads();
+  }
+
+  auto fill_values = [&](int base, float* buf) {  // values that need a conversion or an activation first
+    const int n = min(R, t1 - base);
+    float* vs = buf + planes * R * DP;
+    for (int idx = tid; idx < n * C; idx += TILE_THREADS) {
+      const int r = idx / C, c = blockIdx.x * C + idx % C;
+      if (c >= p.vdim) continue;
+      const float v = ld_any(p.proj, p.proj_dtype, (size_t)(base + r) * p.ld + p.v_off + (size_t)head * p.vdim + c);
+      vs[idx] = p.act == 1 ? v / (1.f + expf(-v)) : v;
+    }
+  };
+  auto stage_round = [&](int base, float* buf) {
+    const int n = min(R, t1 - base);
+    // SLICES threads a row of one plane
+#pragma unroll
+    for (int pl = 0; pl < planes; ++pl)
+      for (int r = tid / SLICES; r < n; r += TILE_THREADS / SLICES) {
+        float* dst = buf + (pl * R + r) * DP;
+        const float* src = per_token ? rows + (size_t)(base + r) * p.ld + (pl == 0 ? p.q_off : p.k_off) + group0
+                                     : p.ready + ((size_t)(base + r) * planes + pl) * hd + head * p.dim;
+#pragma unroll
+        for (int q = 0; q < QUADS; ++q) {
+          const int i = q * SLICES * 4 + (tid % SLICES) * 4;
+          if (wide) {
+            if (i < p.dim) cp_async16(dst + i, src + i);
+          } else {
+            for (int e = 0; e < 4; ++e)
+              if (i + e < p.dim) cp_async4(dst + i + e, src + i + e);
+          }
+        }
+      }
+    float* vs = buf + planes * R * DP;
+    if (v_async) {
+      const float* src = rows + p.v_off + (size_t)head * p.vdim + blockIdx.x * C;
+      for (int idx = tid; idx < n * (C / 4); idx += TILE_THREADS) {
+        const int r = idx / (C / 4), c = (idx % (C / 4)) * 4, left = p.vdim - (int)blockIdx.x * C - c;
+        if (v_wide) {
+          if (left > 0) cp_async16(vs + r * C + c, src + (size_t)(base + r) * p.ld + c);
+        } else {
+          for (int e = 0; e < min(4, left); ++e) cp_async4(vs + r * C + c + e, src + (size_t)(base + r) * p.ld + c + e);
+        }
+      }
+    } else {
+      fill_values(base, buf);
+    }
+    if (per_token && tid < 2 * n)
+      cp_async4(vs + R * C + (tid & 1) * R + (tid >> 1), p.steps + ((size_t)(base + (tid >> 1)) * 2 + (tid & 1)) * p.H + head);
+  };
+
+  auto compute = [&](int base, const float* buf) {
+    const int n = min(R, t1 - base);
+    const float* vs = buf + planes * R * DP + cg * 4;
+    const float* steps = buf + planes * R * DP + R * C;
+    const float* qs = buf + slice * 4;
+#pragma unroll
+    for (int r0 = 0; r0 < R; r0 += BATCH) {
+      if (r0 >= n) break;
+      float acc[BATCH * 4];
+#pragma unroll
+      for (int k = 0; k < BATCH; ++k) {
+        const int r = r0 + k;
+        float o[4] = {0.f, 0.f, 0.f, 0.f};
+        if (r < n) {
+          const float4 v4 = *reinterpret_cast<const float4*>(vs + r * C);
+          float v[4] = {v4.x, v4.y, v4.z, v4.w};
+          float a_all = decay;
+          if (per_token) {
+            const float step = steps[r];
+            a_all = steps[R + r];
+#pragma unroll
+            for (int c = 0; c < 4; ++c) v[c] *= step;
+          }
+#pragma unroll
+          for (int q = 0; q < QUADS; ++q) {
+            const float* at = qs + r * DP + q * SLICES * 4;
+            const float4 q4 = *reinterpret_cast<const float4*>(at), b4 = *reinterpret_cast<const float4*>(at + R * DP);
+            float4 a4 = make_float4(a_all, a_all, a_all, a_all);
+            if (gate) a4 = *reinterpret_cast<const float4*>(at + 2 * R * DP);
+            const float qe[4] = {q4.x, q4.y, q4.z, q4.w}, be[4] = {b4.x, b4.y, b4.z, b4.w}, ae[4] = {a4.x, a4.y, a4.z, a4.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+#pragma unroll
+              for (int c = 0; c < 4; ++c) {
+                S[q * 4 + e][c] = fmaf(ae[e], S[q * 4 + e][c], be[e] * v[c]);
+                o[c] = fmaf(S[q * 4 + e][c], qe[e], o[c]);
+              }
+          }
+        }
+#pragma unroll
+        for (int c = 0; c < 4; ++c) acc[k * 4 + c] = o[c];
+      }
+      // sums over the slices: each exchange leaves a lane half of its values; lane `slice` ends with values
+      // slice * PER .. + PER - 1 of the BATCH * 4 (value k * 4 + c: token k, column c)
+      constexpr int PER = BATCH * 4 / SLICES;
+#pragma unroll
+      for (int o = SLICES / 2, m = BATCH * 2; o > 0; o >>= 1, m >>= 1) {
+        const bool upper = (lane & o) != 0;
+#pragma unroll
+        for (int i = 0; i < BATCH * 2; ++i)
+          if (i < m) {
+            const float keep = upper ? acc[i + m] : acc[i], give = upper ? acc[i] : acc[i + m];
+            acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+          }
+      }
+#pragma unroll
+      for (int i = 0; i < PER; ++i) {
+        const int at = slice * PER + i, r = r0 + (at >> 2), c = at & 3;
+        if (r < n && col0 + c < p.vdim) {
+          float y = acc[i];
+          if (per_token) y = fmaf(skip, vs[r * C + c], y);
+          p.out[(size_t)(base + r) * p.ldo + (size_t)head * p.vdim + col0 + c] = y;
+        }
+      }
+    }
+  };
+
+  if (streamed) {
+    for (int s = 0; s < TILE_STAGES - 1; ++s) {
+      if (t0 + s * R < t1) stage_round(t0 + s * R, tile_smem + s * L::stage);
+      asm volatile("cp.async.commit_group;\n");
+    }
+    int turn = 0;
+    for (int base = t0; base < t1; base += R, turn = (turn + 1) % TILE_STAGES) {
+      float* buf = tile_smem + turn * L::stage;
+      asm volatile("cp.async.wait_group %0;\n" ::"n"(TILE_STAGES - 2));
+      __syncthreads();  // this round has landed for everyone; the round before has been read by everyone
+      const int ahead = base + (TILE_STAGES - 1) * R;
+      if (ahead < t1) stage_round(ahead, tile_smem + ((turn + TILE_STAGES - 1) % TILE_STAGES) * L::stage);
+      asm volatile("cp.async.commit_group;\n");
+      if (v_async && p.act == 1) {  // the activation of the values, in place
+        float* vs = buf + planes * R * DP;
+        for (int idx = tid; idx < R * C; idx += TILE_THREADS) vs[idx] = vs[idx] / (1.f + expf(-vs[idx]));
+        __syncthreads();
+      }
+      compute(base, buf);
+    }
+    asm volatile("cp.async.wait_group 0;\n");
+  } else {
+    for (int base = t0; base < t1; base += R) {
+      const int n = min(R, t1 - base);
+      __syncthreads();
+      if (per_token) {
+        stage_round(base, tile_smem);
+        asm volatile("cp.async.commit_group;\n");
+        asm volatile("cp.async.wait_group 0;\n");
+        __syncthreads();
+        compute(base, tile_smem);
+        continue;
+      }
+      for (int idx = tid; idx < n * p.dim; idx += TILE_THREADS) {
+        const int r = idx / p.dim, i = idx % p.dim;
+        float qv, bv, av;
+        transform(p, base + r, head, i, qv, bv, av);
+        tile_smem[r * DP + i] = qv;
+        tile_smem[(R + r) * DP + i] = bv;
+        if (gate) tile_smem[(2 * R + r) * DP + i] = av;
+      }
+      fill_values(base, tile_smem);
+      __syncthreads();
+      compute(base, tile_smem);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < QUADS * 4; ++k) {
+    const int i = (k >> 2) * (SLICES * 4) + slice * 4 + (k & 3);
+    if (i >= p.dim || col0 >= p.vdim) continue;
+    float* dst = sp + (size_t)i * p.vdim + col0;
+    if (s_wide) {
+      *reinterpret_cast<float4*>(dst) = make_float4(S[k][0], S[k][1], S[k][2], S[k][3]);
+    } else {
+#pragma unroll
+      for (int c = 0; c < 4; ++c)
+        if (col0 + c < p.vdim) dst[c] = S[k][c];
+    }
+  }
+}
+
+template <int SLICES, int QUADS, int KIND>
+int launch_tile_kind(const RecurrenceArgs& a, int S, cudaStream_t stream) {
+  using L = Tile<SLICES, QUADS, KIND>;
+  static bool configured = false;
+  if (!configured) {
+    DSP_CUDA(cudaFuncSetAttribute(recurrence_tile_kernel<SLICES, QUADS, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                  (int)L::smem(TILE_STAGES)));
+    configured = true;
+  }
+  recurrence_tile_kernel<SLICES, QUADS, KIND><<<dim3((a.vdim + L::cols - 1) / L::cols, a.H, S), TILE_THREADS,
+                                                L::smem(a.streamed ? TILE_STAGES : 1), stream>>>(a);
+  DSP_CHECK_LAUNCH("dsp_linear_recurrence");
+  return 0;
+}
+
+template <int SLICES, int QUADS>
+int launch_tile(const RecurrenceArgs& a, int S, cudaStream_t stream) {
+  if (a.mode == STEP_DECAY) return launch_tile_kind<SLICES, QUADS, TOKEN_DECAY>(a, S, stream);
+  if (a.mode == FIXED_DECAY) return launch_tile_kind<SLICES, QUADS, SCALAR_DECAY>(a, S, stream);
+  return launch_tile_kind<SLICES, QUADS, VECTOR_DECAY>(a, S, stream);
+}
+
 template <int ROWS, int TPR, int KIND>
 int launch_kind(const RecurrenceArgs& a, int S, size_t smem, cudaStream_t stream) {
   static size_t configured = 48 * 1024;
@@ -421,21 +687,20 @@ extern "C" int dsp_linear_recurrence(const void* proj, int proj_dtype, long ld, 
   a.steps = steps; a.skip = skip; a.heads_per_group = mode == STEP_DECAY ? heads_per_group : 1;
   a.state = state; a.state_slot = state_slot; a.q_start = q_start; a.positions = positions;
   a.out = out; a.ldo = ldo; a.ready = scratch;
-  // threads per column: as many as bring a thread's state rows down to 8 (a power of two, at
-  // most a warp); beyond 256 rows a thread holds 16 or 32
-  int slices = 1;
-  while (slices < 32 && (dim + slices - 1) / slices > 8) slices *= 2;
-  const int rows = (dim + slices - 1) / slices;
+  a.streamed = scratch != nullptr || (mode == STEP_DECAY && T > 2 * S);
+  // one column a thread, 32 threads a column, 16 or 32 state rows a thread (beyond 256 state rows)
+  const bool tiled = dim <= 256;
+  const int slices = 32, rows = (dim + slices - 1) / slices;
   a.slices = slices;
   a.cols_per_block = THREADS / slices;
-  const int R = rows <= 8 ? 8 : (rows <= 16 ? 16 : 32);
+  const int R = rows <= 16 ? 16 : 32;
   const int dpad = slices * R;
-  a.tokens_per_round = dpad <= 256 ? 16 : 8;
+  a.tokens_per_round = 8;
   const int planes = mode == FORGET_GATE || mode == KEY_DECAY ? 3 : 2;
   const size_t buf = (size_t)planes * a.tokens_per_round * dpad + (size_t)a.tokens_per_round * a.cols_per_block +
                      (mode == STEP_DECAY ? 2 * a.tokens_per_round : 0);
   const size_t smem = sizeof(float) * ((scratch || mode == STEP_DECAY ? 2 : 1) * buf + (size_t)a.tokens_per_round * a.cols_per_block);
-  DSP_REQUIRE(smem <= 227 * 1024, "dsp_linear_recurrence: state rows of %d do not fit shared memory", dim);
+  DSP_REQUIRE(tiled || smem <= 227 * 1024, "dsp_linear_recurrence: state rows of %d do not fit shared memory", dim);
   if (scratch && mode == KEY_DECAY) {
     const unsigned tiles = (unsigned)((H * dim + 255) / 256);
     DSP_REQUIRE(tiles <= 65535, "dsp_linear_recurrence: %d heads of %d are too many", H, dim);
@@ -448,12 +713,10 @@ extern "C" int dsp_linear_recurrence(const void* proj, int proj_dtype, long ld, 
     recurrence_prepare_kernel<<<(unsigned)(want < cap ? want : cap), 256, 0, stream>>>(a, T);
     DSP_CHECK_LAUNCH("dsp_linear_recurrence (first kernel)");
   }
-  if (a.tokens_per_round == 16) {
-    if (R == 8) return launch<8, 16>(a, S, smem, stream);
-    if (R == 16) return launch<16, 16>(a, S, smem, stream);
-    return launch<32, 16>(a, S, smem, stream);
-  }
-  if (R == 8) return launch<8, 8>(a, S, smem, stream);
+  if (dim <= 32) return launch_tile<8, 1>(a, S, stream);
+  if (dim <= 64) return launch_tile<16, 1>(a, S, stream);
+  if (dim <= 128) return launch_tile<32, 1>(a, S, stream);
+  if (tiled) return launch_tile<32, 2>(a, S, stream);
   if (R == 16) return launch<16, 8>(a, S, smem, stream);
   return launch<32, 8>(a, S, smem, stream);
 }
