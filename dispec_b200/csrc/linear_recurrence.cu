@@ -33,6 +33,8 @@
 // are staged, in one kernel.  State rows beyond 256 take a kernel of their own with one column a
 // thread.  A request whose first row carries a negative position (a padding row of a captured step) is
 // skipped: its state slot belongs to someone else.
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace {
@@ -366,6 +368,25 @@ linear_recurrence_kernel(const RecurrenceArgs p) {
   }
 }
 
+// Two 32-bit floats side by side: one instruction, each half rounded as its scalar form is.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2f(float a, float b) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ void unpack2f(f32x2 v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
 // The kernel for up to 256 state rows.  SLICES lanes times QUADS times four rows cover the state's rows.
 constexpr int TILE_WARPS = 4, TILE_THREADS = 32 * TILE_WARPS, TILE_STAGES = 4, BATCH = 8;
 
@@ -404,21 +425,27 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
   // state rows q * SLICES * 4 + slice * 4 + e (e < 4) of columns col0 .. col0 + 3
   float* sp = p.state + (((size_t)p.state_slot[seq] * p.H + head) * p.dim) * p.vdim;
   const bool s_wide = p.vdim % 4 == 0;
-  float S[QUADS * 4][4];
+  auto row_of = [&](int k) { return (k >> 2) * (SLICES * 4) + slice * 4 + (k & 3); };
+  f32x2 S[QUADS * 2][4];  // [pair of rows 2k, 2k + 1][column]
 #pragma unroll
-  for (int k = 0; k < QUADS * 4; ++k) {
-    const int i = (k >> 2) * (SLICES * 4) + slice * 4 + (k & 3);
-    S[k][0] = S[k][1] = S[k][2] = S[k][3] = 0.f;
-    if (i >= p.dim || col0 >= p.vdim) continue;
-    const float* src = sp + (size_t)i * p.vdim + col0;
-    if (s_wide) {
-      const float4 v = *reinterpret_cast<const float4*>(src);
-      S[k][0] = v.x, S[k][1] = v.y, S[k][2] = v.z, S[k][3] = v.w;
-    } else {
+  for (int k = 0; k < QUADS * 2; ++k) {
+    float s[2][4] = {};
 #pragma unroll
-      for (int c = 0; c < 4; ++c)
-        if (col0 + c < p.vdim) S[k][c] = src[c];
+    for (int h = 0; h < 2; ++h) {
+      const int i = row_of(2 * k + h);
+      if (i >= p.dim || col0 >= p.vdim) continue;
+      const float* src = sp + (size_t)i * p.vdim + col0;
+      if (s_wide) {
+        const float4 v = *reinterpret_cast<const float4*>(src);
+        s[h][0] = v.x, s[h][1] = v.y, s[h][2] = v.z, s[h][3] = v.w;
+      } else {
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+          if (col0 + c < p.vdim) s[h][c] = src[c];
+      }
     }
+#pragma unroll
+    for (int c = 0; c < 4; ++c) S[k][c] = pack2f(s[0][c], s[1][c]);
   }
   const float decay = KIND == SCALAR_DECAY ? p.decay[head] : 0.f;
   const float skip = per_token ? p.skip[head] : 0.f;
@@ -477,8 +504,10 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
       cp_async4(vs + R * C + (tid & 1) * R + (tid >> 1), p.steps + ((size_t)(base + (tid >> 1)) * 2 + (tid & 1)) * p.H + head);
   };
 
-  auto compute = [&](int base, const float* buf) {
-    const int n = min(R, t1 - base);
+  // one round; `full`: all of its tokens are there (no conditions between the tokens' loads)
+  auto compute_round = [&](auto full, int base, const float* buf) {
+    constexpr bool whole_round = decltype(full)::value;
+    const int n = whole_round ? R : min(R, t1 - base);
     const float* vs = buf + planes * R * DP + cg * 4;
     const float* steps = buf + planes * R * DP + R * C;
     const float* qs = buf + slice * 4;
@@ -490,7 +519,7 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
       for (int k = 0; k < BATCH; ++k) {
         const int r = r0 + k;
         float o[4] = {0.f, 0.f, 0.f, 0.f};
-        if (r < n) {
+        if (whole_round || r < n) {
           const float4 v4 = *reinterpret_cast<const float4*>(vs + r * C);
           float v[4] = {v4.x, v4.y, v4.z, v4.w};
           float a_all = decay;
@@ -500,20 +529,31 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
 #pragma unroll
             for (int c = 0; c < 4; ++c) v[c] *= step;
           }
+          f32x2 v2[4], o2[4];
+#pragma unroll
+          for (int c = 0; c < 4; ++c) v2[c] = pack2f(v[c], v[c]);
+          const f32x2 all2 = pack2f(a_all, a_all);
 #pragma unroll
           for (int q = 0; q < QUADS; ++q) {
             const float* at = qs + r * DP + q * SLICES * 4;
-            const float4 q4 = *reinterpret_cast<const float4*>(at), b4 = *reinterpret_cast<const float4*>(at + R * DP);
-            float4 a4 = make_float4(a_all, a_all, a_all, a_all);
-            if (gate) a4 = *reinterpret_cast<const float4*>(at + 2 * R * DP);
-            const float qe[4] = {q4.x, q4.y, q4.z, q4.w}, be[4] = {b4.x, b4.y, b4.z, b4.w}, ae[4] = {a4.x, a4.y, a4.z, a4.w};
+            const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(at), b4 = *reinterpret_cast<const ulonglong2*>(at + R * DP);
+            ulonglong2 a4 = make_ulonglong2(all2, all2);
+            if (gate) a4 = *reinterpret_cast<const ulonglong2*>(at + 2 * R * DP);
+            const f32x2 qe[2] = {q4.x, q4.y}, be[2] = {b4.x, b4.y}, ae[2] = {a4.x, a4.y};
 #pragma unroll
-            for (int e = 0; e < 4; ++e)
+            for (int e = 0; e < 2; ++e)
 #pragma unroll
               for (int c = 0; c < 4; ++c) {
-                S[q * 4 + e][c] = fmaf(ae[e], S[q * 4 + e][c], be[e] * v[c]);
-                o[c] = fmaf(S[q * 4 + e][c], qe[e], o[c]);
+                f32x2& s = S[q * 2 + e][c];
+                s = fma2(ae[e], s, mul2(be[e], v2[c]));
+                o2[c] = q == 0 && e == 0 ? mul2(s, qe[e]) : fma2(s, qe[e], o2[c]);
               }
+          }
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            float even, odd;
+            unpack2f(o2[c], even, odd);
+            o[c] = even + odd;
           }
         }
 #pragma unroll
@@ -535,13 +575,20 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
 #pragma unroll
       for (int i = 0; i < PER; ++i) {
         const int at = slice * PER + i, r = r0 + (at >> 2), c = at & 3;
-        if (r < n && col0 + c < p.vdim) {
+        if ((whole_round || r < n) && col0 + c < p.vdim) {
           float y = acc[i];
           if (per_token) y = fmaf(skip, vs[r * C + c], y);
           p.out[(size_t)(base + r) * p.ldo + (size_t)head * p.vdim + col0 + c] = y;
         }
       }
     }
+  };
+
+  auto compute = [&](int base, const float* buf) {
+    if (base + R <= t1)
+      compute_round(std::true_type{}, base, buf);
+    else
+      compute_round(std::false_type{}, base, buf);
   };
 
   if (streamed) {
@@ -591,16 +638,22 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
     }
   }
 #pragma unroll
-  for (int k = 0; k < QUADS * 4; ++k) {
-    const int i = (k >> 2) * (SLICES * 4) + slice * 4 + (k & 3);
-    if (i >= p.dim || col0 >= p.vdim) continue;
-    float* dst = sp + (size_t)i * p.vdim + col0;
-    if (s_wide) {
-      *reinterpret_cast<float4*>(dst) = make_float4(S[k][0], S[k][1], S[k][2], S[k][3]);
-    } else {
+  for (int k = 0; k < QUADS * 2; ++k) {
+    float s[2][4];
 #pragma unroll
-      for (int c = 0; c < 4; ++c)
-        if (col0 + c < p.vdim) dst[c] = S[k][c];
+    for (int c = 0; c < 4; ++c) unpack2f(S[k][c], s[0][c], s[1][c]);
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int i = row_of(2 * k + h);
+      if (i >= p.dim || col0 >= p.vdim) continue;
+      float* dst = sp + (size_t)i * p.vdim + col0;
+      if (s_wide) {
+        *reinterpret_cast<float4*>(dst) = make_float4(s[h][0], s[h][1], s[h][2], s[h][3]);
+      } else {
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+          if (col0 + c < p.vdim) dst[c] = s[h][c];
+      }
     }
   }
 }
