@@ -21,11 +21,12 @@
 //                 token and head and the value scaled by another (`steps`); o_t gets skip[head] * v_t on top:
 //                     S_t = a S_(t-1) + step b_t v_t^T,   o_t = S_t^T q_t + skip v_t
 //
-// One block of four warps per (request, head, tile of value columns); what a block computes is
-// sequential in the tokens of its request.  A thread holds a tile of the state in registers, four
-// neighbouring rows (twice four beyond 128 rows) of four neighbouring columns, so that what it
-// reads of q, b and a serves four columns and what it reads of v serves four rows.  The SLICES lanes
-// that share columns cover the rows; eight tokens' partial outputs are added over them together, each
+// One block of eight warps per (request, head, tile of value columns); what a block computes is
+// sequential in the tokens of its request.  A thread holds a tile of the state in registers, two (or
+// four) neighbouring rows of four neighbouring columns, so that what it reads of q, b and a serves four
+// columns; rows go through the multipliers in pairs.  The SLICES lanes that share columns cover the rows
+// (beyond 64 rows two groups of warps do: an SM has two warps a scheduler to hide one another's latencies
+// even when a lone prompt leaves it one block); eight tokens' partial outputs are added over them together, each
 // exchange halving the values a lane still holds, and end up one to a lane.  Tokens are staged through shared
 // memory in rounds: for portions of prompts a first, fully parallel kernel writes q_t, b_t (and a_t) of
 // every token as floats (STEP_DECAY streams its rows as they are), and the recurrence streams them in
@@ -116,7 +117,13 @@ __device__ __forceinline__ void transform(const RecurrenceArgs& p, int token, in
     bv = ld_any(p.proj, p.proj_dtype, ko + i) * p.key_scale;
     const int c = head * p.dim + i, hd = p.H * p.dim;
     float z = p.gate_bias[c];
-    for (int r = 0; r < p.rank; ++r) z = fmaf(p.gate_map[(size_t)r * hd + c], ld_any(p.proj, p.proj_dtype, rowp + p.low_off + r), z);
+    if (p.proj_dtype == DSP_F32) {
+      const float* low = reinterpret_cast<const float*>(p.proj) + rowp + p.low_off;
+#pragma unroll 8
+      for (int r = 0; r < p.rank; ++r) z = fmaf(p.gate_map[(size_t)r * hd + c], low[r], z);
+    } else {
+      for (int r = 0; r < p.rank; ++r) z = fmaf(p.gate_map[(size_t)r * hd + c], ld_any(p.proj, p.proj_dtype, rowp + p.low_off + r), z);
+    }
     av = sigmoid_power(z, p.power);
   } else {
     const float rq = ld_any(p.proj, p.proj_dtype, qo + i);
@@ -387,24 +394,28 @@ __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
   return r;
 }
 
-// The kernel for up to 256 state rows.  SLICES lanes times QUADS times four rows cover the state's rows.
-constexpr int TILE_WARPS = 4, TILE_THREADS = 32 * TILE_WARPS, TILE_STAGES = 4, BATCH = 8;
+// The kernel for up to 256 state rows.  SLICES lanes, PAIRS pairs of rows a lane and PARTS groups of warps cover
+// the state's rows (padded); with two groups every output is the sum of two warps' results, which meet in
+// shared memory and leave for the result one round later.
+constexpr int TILE_WARPS = 8, TILE_THREADS = 32 * TILE_WARPS, TILE_STAGES = 4, BATCH = 8;
 
-template <int SLICES, int QUADS, int KIND>
+template <int SLICES, int PAIRS, int PARTS, int KIND>
 struct Tile {
   static constexpr bool gate = KIND == VECTOR_DECAY, per_token = KIND == TOKEN_DECAY;
   static constexpr int planes = gate ? 3 : 2;
-  static constexpr int rows = SLICES * 4 * QUADS;                     // state rows, padded
-  static constexpr int cols = TILE_WARPS * (32 / SLICES) * 4;         // value columns of a block
-  static constexpr int round = QUADS == 1 ? 16 : 8;                   // tokens staged together
+  static constexpr int part_rows = SLICES * 2 * PAIRS;                       // state rows of a group of warps
+  static constexpr int rows = part_rows * PARTS;                             // state rows, padded
+  static constexpr int cols = TILE_WARPS / PARTS * (32 / SLICES) * 4;        // value columns of a block
+  static constexpr int round = rows <= 128 ? 16 : 8;                         // tokens staged together
   static constexpr int stage = planes * round * rows + round * cols + (per_token ? 2 * round : 0);
-  static constexpr size_t smem(int stages) { return sizeof(float) * stages * stage; }
+  static constexpr int meet = PARTS == 1 ? 0 : 2 * PARTS * round * cols;     // results of two rounds
+  static constexpr size_t smem(int stages) { return sizeof(float) * (stages * stage + meet); }
 };
 
-template <int SLICES, int QUADS, int KIND>
-__global__ void __launch_bounds__(TILE_THREADS)
+template <int SLICES, int PAIRS, int PARTS, int KIND>
+__global__ void __launch_bounds__(TILE_THREADS, 2)
 recurrence_tile_kernel(const RecurrenceArgs p) {
-  using L = Tile<SLICES, QUADS, KIND>;
+  using L = Tile<SLICES, PAIRS, PARTS, KIND>;
   constexpr bool gate = L::gate, per_token = L::per_token;
   constexpr int DP = L::rows, C = L::cols, R = L::round, planes = L::planes;
   extern __shared__ __align__(16) float tile_smem[];
@@ -412,7 +423,9 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
   const int t0 = p.q_start[seq], t1 = p.q_start[seq + 1];
   if (t1 <= t0 || p.positions[t0] < 0) return;
   const int tid = threadIdx.x, lane = tid & 31, slice = lane % SLICES;
-  const int cg = (tid >> 5) * (32 / SLICES) + lane / SLICES;  // this thread's group of four columns
+  constexpr int PART_WARPS = TILE_WARPS / PARTS;
+  const int part = (tid >> 5) / PART_WARPS;  // this warp's group of state rows
+  const int cg = (tid >> 5) % PART_WARPS * (32 / SLICES) + lane / SLICES;  // this thread's group of four columns
   const int col0 = blockIdx.x * C + cg * 4;
   const bool streamed = p.streamed != 0;
   const float* rows = reinterpret_cast<const float*>(p.proj);
@@ -422,17 +435,17 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
   const bool v_wide = whole && p.v_off % 4 == 0 && p.vdim % 4 == 0;
   const int hd = p.H * p.dim, group0 = (head / p.heads_per_group) * p.dim;
 
-  // state rows q * SLICES * 4 + slice * 4 + e (e < 4) of columns col0 .. col0 + 3
+  // 2 PAIRS neighbouring state rows of columns col0 .. col0 + 3
   float* sp = p.state + (((size_t)p.state_slot[seq] * p.H + head) * p.dim) * p.vdim;
   const bool s_wide = p.vdim % 4 == 0;
-  auto row_of = [&](int k) { return (k >> 2) * (SLICES * 4) + slice * 4 + (k & 3); };
-  f32x2 S[QUADS * 2][4];  // [pair of rows 2k, 2k + 1][column]
+  const int row0 = part * L::part_rows + slice * 2 * PAIRS;
+  f32x2 S[PAIRS][4];  // [pair of rows 2k, 2k + 1][column]
 #pragma unroll
-  for (int k = 0; k < QUADS * 2; ++k) {
+  for (int k = 0; k < PAIRS; ++k) {
     float s[2][4] = {};
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
-      const int i = row_of(2 * k + h);
+      const int i = row0 + 2 * k + h;
       if (i >= p.dim || col0 >= p.vdim) continue;
       const float* src = sp + (size_t)i * p.vdim + col0;
       if (s_wide) {
@@ -468,16 +481,15 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
   };
   auto stage_round = [&](int base, float* buf) {
     const int n = min(R, t1 - base);
-    // SLICES threads a row of one plane
+    constexpr int ROW_THREADS = DP / 4 < 32 ? DP / 4 : 32;  // threads a row of one plane
 #pragma unroll
     for (int pl = 0; pl < planes; ++pl)
-      for (int r = tid / SLICES; r < n; r += TILE_THREADS / SLICES) {
+      for (int r = tid / ROW_THREADS; r < n; r += TILE_THREADS / ROW_THREADS) {
         float* dst = buf + (pl * R + r) * DP;
         const float* src = per_token ? rows + (size_t)(base + r) * p.ld + (pl == 0 ? p.q_off : p.k_off) + group0
                                      : p.ready + ((size_t)(base + r) * planes + pl) * hd + head * p.dim;
 #pragma unroll
-        for (int q = 0; q < QUADS; ++q) {
-          const int i = q * SLICES * 4 + (tid % SLICES) * 4;
+        for (int i = (tid % ROW_THREADS) * 4; i < DP; i += ROW_THREADS * 4) {
           if (wide) {
             if (i < p.dim) cp_async16(dst + i, src + i);
           } else {
@@ -504,13 +516,16 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
       cp_async4(vs + R * C + (tid & 1) * R + (tid >> 1), p.steps + ((size_t)(base + (tid >> 1)) * 2 + (tid & 1)) * p.H + head);
   };
 
+  float* meet = tile_smem + (streamed ? TILE_STAGES : 1) * L::stage;
+  int turn2 = 0;  // which of the two meeting places the latest round used
   // one round; `full`: all of its tokens are there (no conditions between the tokens' loads)
   auto compute_round = [&](auto full, int base, const float* buf) {
     constexpr bool whole_round = decltype(full)::value;
     const int n = whole_round ? R : min(R, t1 - base);
     const float* vs = buf + planes * R * DP + cg * 4;
     const float* steps = buf + planes * R * DP + R * C;
-    const float* qs = buf + slice * 4;
+    const float* qs = buf + row0;
+    float* mine = meet + ((turn2 * PARTS + part) * R) * C + cg * 4;  // (two groups of warps only)
 #pragma unroll
     for (int r0 = 0; r0 < R; r0 += BATCH) {
       if (r0 >= n) break;
@@ -534,20 +549,15 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
           for (int c = 0; c < 4; ++c) v2[c] = pack2f(v[c], v[c]);
           const f32x2 all2 = pack2f(a_all, a_all);
 #pragma unroll
-          for (int q = 0; q < QUADS; ++q) {
-            const float* at = qs + r * DP + q * SLICES * 4;
-            const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(at), b4 = *reinterpret_cast<const ulonglong2*>(at + R * DP);
-            ulonglong2 a4 = make_ulonglong2(all2, all2);
-            if (gate) a4 = *reinterpret_cast<const ulonglong2*>(at + 2 * R * DP);
-            const f32x2 qe[2] = {q4.x, q4.y}, be[2] = {b4.x, b4.y}, ae[2] = {a4.x, a4.y};
+          for (int e = 0; e < PAIRS; ++e) {
+            const f32x2* at = reinterpret_cast<const f32x2*>(qs + r * DP) + e;
+            const f32x2 qe = at[0], be = at[R * DP / 2], ae = gate ? at[R * DP] : all2;
 #pragma unroll
-            for (int e = 0; e < 2; ++e)
-#pragma unroll
-              for (int c = 0; c < 4; ++c) {
-                f32x2& s = S[q * 2 + e][c];
-                s = fma2(ae[e], s, mul2(be[e], v2[c]));
-                o2[c] = q == 0 && e == 0 ? mul2(s, qe[e]) : fma2(s, qe[e], o2[c]);
-              }
+            for (int c = 0; c < 4; ++c) {
+              f32x2& s = S[e][c];
+              s = fma2(ae, s, mul2(be, v2[c]));
+              o2[c] = e == 0 ? mul2(s, qe) : fma2(s, qe, o2[c]);
+            }
           }
 #pragma unroll
           for (int c = 0; c < 4; ++c) {
@@ -577,18 +587,37 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
         const int at = slice * PER + i, r = r0 + (at >> 2), c = at & 3;
         if ((whole_round || r < n) && col0 + c < p.vdim) {
           float y = acc[i];
-          if (per_token) y = fmaf(skip, vs[r * C + c], y);
-          p.out[(size_t)(base + r) * p.ldo + (size_t)head * p.vdim + col0 + c] = y;
+          if (per_token && part == 0) y = fmaf(skip, vs[r * C + c], y);
+          if (PARTS > 1)
+            mine[r * C + c] = y;
+          else
+            p.out[(size_t)(base + r) * p.ldo + (size_t)head * p.vdim + col0 + c] = y;
         }
       }
     }
   };
 
   auto compute = [&](int base, const float* buf) {
+    turn2 ^= 1;
     if (base + R <= t1)
       compute_round(std::true_type{}, base, buf);
     else
       compute_round(std::false_type{}, base, buf);
+  };
+
+  // the results of the round at `base` that two groups of warps left (called behind a barrier)
+  auto flush = [&](int base) {
+    if constexpr (PARTS > 1) {
+      const int n = min(R, t1 - base);
+      const float* r0 = meet + turn2 * PARTS * R * C;
+      for (int idx = tid; idx < n * C; idx += TILE_THREADS) {
+        const int c = blockIdx.x * C + idx % C;
+        float y = r0[idx];
+#pragma unroll
+        for (int k = 1; k < PARTS; ++k) y += r0[k * R * C + idx];
+        if (c < p.vdim) p.out[(size_t)(base + idx / C) * p.ldo + (size_t)head * p.vdim + c] = y;
+      }
+    }
   };
 
   if (streamed) {
@@ -601,6 +630,7 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
       float* buf = tile_smem + turn * L::stage;
       asm volatile("cp.async.wait_group %0;\n" ::"n"(TILE_STAGES - 2));
       __syncthreads();  // this round has landed for everyone; the round before has been read by everyone
+      if (base > t0) flush(base - R);
       const int ahead = base + (TILE_STAGES - 1) * R;
       if (ahead < t1) stage_round(ahead, tile_smem + ((turn + TILE_STAGES - 1) % TILE_STAGES) * L::stage);
       asm volatile("cp.async.commit_group;\n");
@@ -616,6 +646,7 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
     for (int base = t0; base < t1; base += R) {
       const int n = min(R, t1 - base);
       __syncthreads();
+      if (base > t0) flush(base - R);
       if (per_token) {
         stage_round(base, tile_smem);
         asm volatile("cp.async.commit_group;\n");
@@ -637,14 +668,18 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
       compute(base, tile_smem);
     }
   }
+  if (PARTS > 1) {
+    __syncthreads();
+    flush(t0 + (t1 - t0 - 1) / R * R);
+  }
 #pragma unroll
-  for (int k = 0; k < QUADS * 2; ++k) {
+  for (int k = 0; k < PAIRS; ++k) {
     float s[2][4];
 #pragma unroll
     for (int c = 0; c < 4; ++c) unpack2f(S[k][c], s[0][c], s[1][c]);
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
-      const int i = row_of(2 * k + h);
+      const int i = row0 + 2 * k + h;
       if (i >= p.dim || col0 >= p.vdim) continue;
       float* dst = sp + (size_t)i * p.vdim + col0;
       if (s_wide) {
@@ -658,26 +693,26 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
   }
 }
 
-template <int SLICES, int QUADS, int KIND>
+template <int SLICES, int PAIRS, int PARTS, int KIND>
 int launch_tile_kind(const RecurrenceArgs& a, int S, cudaStream_t stream) {
-  using L = Tile<SLICES, QUADS, KIND>;
+  using L = Tile<SLICES, PAIRS, PARTS, KIND>;
   static bool configured = false;
   if (!configured) {
-    DSP_CUDA(cudaFuncSetAttribute(recurrence_tile_kernel<SLICES, QUADS, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    DSP_CUDA(cudaFuncSetAttribute(recurrence_tile_kernel<SLICES, PAIRS, PARTS, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                   (int)L::smem(TILE_STAGES)));
     configured = true;
   }
-  recurrence_tile_kernel<SLICES, QUADS, KIND><<<dim3((a.vdim + L::cols - 1) / L::cols, a.H, S), TILE_THREADS,
-                                                L::smem(a.streamed ? TILE_STAGES : 1), stream>>>(a);
+  recurrence_tile_kernel<SLICES, PAIRS, PARTS, KIND><<<dim3((a.vdim + L::cols - 1) / L::cols, a.H, S), TILE_THREADS,
+                                                       L::smem(a.streamed ? TILE_STAGES : 1), stream>>>(a);
   DSP_CHECK_LAUNCH("dsp_linear_recurrence");
   return 0;
 }
 
-template <int SLICES, int QUADS>
+template <int SLICES, int PAIRS, int PARTS>
 int launch_tile(const RecurrenceArgs& a, int S, cudaStream_t stream) {
-  if (a.mode == STEP_DECAY) return launch_tile_kind<SLICES, QUADS, TOKEN_DECAY>(a, S, stream);
-  if (a.mode == FIXED_DECAY) return launch_tile_kind<SLICES, QUADS, SCALAR_DECAY>(a, S, stream);
-  return launch_tile_kind<SLICES, QUADS, VECTOR_DECAY>(a, S, stream);
+  if (a.mode == STEP_DECAY) return launch_tile_kind<SLICES, PAIRS, PARTS, TOKEN_DECAY>(a, S, stream);
+  if (a.mode == FIXED_DECAY) return launch_tile_kind<SLICES, PAIRS, PARTS, SCALAR_DECAY>(a, S, stream);
+  return launch_tile_kind<SLICES, PAIRS, PARTS, VECTOR_DECAY>(a, S, stream);
 }
 
 template <int ROWS, int TPR, int KIND>
@@ -766,10 +801,10 @@ extern "C" int dsp_linear_recurrence(const void* proj, int proj_dtype, long ld, 
     recurrence_prepare_kernel<<<(unsigned)(want < cap ? want : cap), 256, 0, stream>>>(a, T);
     DSP_CHECK_LAUNCH("dsp_linear_recurrence (first kernel)");
   }
-  if (dim <= 32) return launch_tile<8, 1>(a, S, stream);
-  if (dim <= 64) return launch_tile<16, 1>(a, S, stream);
-  if (dim <= 128) return launch_tile<32, 1>(a, S, stream);
-  if (tiled) return launch_tile<32, 2>(a, S, stream);
+  if (dim <= 32) return launch_tile<16, 1, 1>(a, S, stream);
+  if (dim <= 64) return launch_tile<32, 1, 1>(a, S, stream);
+  if (dim <= 128) return launch_tile<32, 1, 2>(a, S, stream);
+  if (tiled) return launch_tile<32, 2, 2>(a, S, stream);
   if (R == 16) return launch<16, 8>(a, S, smem, stream);
   return launch<32, 8>(a, S, smem, stream);
 }

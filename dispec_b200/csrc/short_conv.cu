@@ -68,6 +68,28 @@ __device__ __forceinline__ float conv_at(const ConvIn& p, const Turn& r, const f
   return acc;
 }
 
+// four neighbouring channels of a token whose taps all lie in the step's rows (floats, 16-byte aligned): the
+// same sums in the same order
+__device__ __forceinline__ float4 conv_at4(const ConvIn& p, const float* row, int c) {
+  const float* u = row + p.off + c - (size_t)(p.taps - 1) * p.ld;
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+  for (int j = 0; j < p.taps; ++j) {
+    const float4 w = *reinterpret_cast<const float4*>(p.w + (size_t)j * p.channels + c);
+    const float4 x = *reinterpret_cast<const float4*>(u + (size_t)j * p.ld);
+    acc.x = fmaf(w.x, x.x, acc.x);
+    acc.y = fmaf(w.y, x.y, acc.y);
+    acc.z = fmaf(w.z, x.z, acc.z);
+    acc.w = fmaf(w.w, x.w, acc.w);
+  }
+  return acc;
+}
+// whether conv_at4 serves token i: not one of those whose taps reach into the state slot
+__device__ __forceinline__ bool in_fours(const ConvIn& p, int i) {
+  return p.w && p.dtype == DSP_F32 && i >= p.taps - 1 && p.channels % 4 == 0 && p.off % 4 == 0 && p.ld % 4 == 0 &&
+         (((uintptr_t)p.u | (uintptr_t)p.w) & 15) == 0;
+}
+
 // leaves the portion's last taps - 1 inputs of channel c in the slot (in place: row m is written before
 // the rows behind it are, and reads rows at or behind m + n)
 __device__ __forceinline__ void keep_inputs(const ConvIn& p, const Turn& r, float* hist, int c) {
@@ -87,14 +109,26 @@ conv_steps_kernel(const ConvIn p, const float* __restrict__ bias, float* __restr
   if (p.positions[t] < 0) return;
   const Turn r = turn_of(p, t);
   float* hist = p.hist + (size_t)p.state_slot[r.seq] * (p.taps - 1) * p.channels;
-  for (int i = r.first; i < r.first + r.count; ++i)
-#pragma unroll
-    for (int k = 0; k < PER_THREAD; ++k) {
-      const int c = (blockIdx.y * PER_THREAD + k) * 256 + threadIdx.x;
-      if (c >= p.channels) break;
-      const float v = conv_at(p, r, hist, c, i) + (bias ? bias[c] : 0.f);
-      out[(size_t)(r.row0 + i) * ldo + c] = v / (1.f + expf(-v));
+  auto silu = [](float v) { return v / (1.f + expf(-v)); };
+  if (!r.owner && r.count == 1 && in_fours(p, r.first) && ldo % 4 == 0 && ((uintptr_t)out & 15) == 0 && ((uintptr_t)bias & 15) == 0) {
+    const int c = (blockIdx.y * 256 + threadIdx.x) * 4;
+    if (c < p.channels) {
+      float4 v = conv_at4(p, reinterpret_cast<const float*>(p.u) + (size_t)t * p.ld, c);
+      if (bias) {
+        const float4 b = *reinterpret_cast<const float4*>(bias + c);
+        v.x += b.x, v.y += b.y, v.z += b.z, v.w += b.w;
+      }
+      *reinterpret_cast<float4*>(out + (size_t)t * ldo + c) = make_float4(silu(v.x), silu(v.y), silu(v.z), silu(v.w));
     }
+  } else {
+    for (int i = r.first; i < r.first + r.count; ++i)
+#pragma unroll
+      for (int k = 0; k < PER_THREAD; ++k) {
+        const int c = (blockIdx.y * PER_THREAD + k) * 256 + threadIdx.x;
+        if (c >= p.channels) break;
+        out[(size_t)(r.row0 + i) * ldo + c] = silu(conv_at(p, r, hist, c, i) + (bias ? bias[c] : 0.f));
+      }
+  }
   if (r.owner)
     for (int k = 0; k < PER_THREAD; ++k) {
       const int c = (blockIdx.y * PER_THREAD + k) * 256 + threadIdx.x;
@@ -113,7 +147,7 @@ qkv_conv_rotate_store_kernel(const ConvIn p, const int* __restrict__ page_table,
                              void* __restrict__ v_pool, int pool_dtype, const float* __restrict__ inv_freq, int rot,
                              int interleaved, int head_norm, float norm_eps, float v_scale, void* __restrict__ q_out,
                              long ld_q, int H, int G, int Dk, int Dv, int page_size, int num_pages, int write_kv, int* err) {
-  extern __shared__ float row[];  // [channels] then [rot/2] cosines, [rot/2] sines
+  extern __shared__ __align__(16) float row[];  // [channels] then [rot/2] cosines, [rot/2] sines
   const int t = blockIdx.x;
   if (p.positions[t] < 0) return;
   const Turn r = turn_of(p, t);
@@ -123,7 +157,11 @@ qkv_conv_rotate_store_kernel(const ConvIn p, const int* __restrict__ page_table,
   const int half = rot / 2, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
   for (int i = r.first; i < r.first + r.count; ++i) {
     const int tok = r.row0 + i, pos = p.positions[tok];
-    for (int c = tid; c < p.channels; c += blockDim.x) row[c] = conv_at(p, r, hist, c, i);
+    if (in_fours(p, i))
+      for (int c = tid * 4; c < p.channels; c += blockDim.x * 4)
+        *reinterpret_cast<float4*>(row + c) = conv_at4(p, reinterpret_cast<const float*>(p.u) + (size_t)tok * p.ld, c);
+    else
+      for (int c = tid; c < p.channels; c += blockDim.x) row[c] = conv_at(p, r, hist, c, i);
     for (int m = tid; m < half; m += blockDim.x) sincosf((float)pos * inv_freq[m], &cs[half + m], &cs[m]);
     __syncthreads();
     const int page = write_kv ? page_table[(size_t)r.seq * pt_stride + pos / page_size] : -1;
