@@ -22,18 +22,18 @@
 //                     S_t = a S_(t-1) + step b_t v_t^T,   o_t = S_t^T q_t + skip v_t
 //
 // One block of eight warps per (request, head, tile of value columns); what a block computes is
-// sequential in the tokens of its request.  A thread holds a tile of the state in registers, two (or
-// four) neighbouring rows of four neighbouring columns, so that what it reads of q, b and a serves four
-// columns; rows go through the multipliers in pairs.  The SLICES lanes that share columns cover the rows
-// (beyond 64 rows two groups of warps do: an SM has two warps a scheduler to hide one another's latencies
-// even when a lone prompt leaves it one block); eight tokens' partial outputs are added over them together, each
-// exchange halving the values a lane still holds, and end up one to a lane.  Tokens are staged through shared
-// memory in rounds: for portions of prompts a first, fully parallel kernel writes q_t, b_t (and a_t) of
-// every token as floats (STEP_DECAY streams its rows as they are), and the recurrence streams them in
-// with cp.async, three rounds ahead of the one that is computed; single tokens are transformed as they
-// are staged, in one kernel.  State rows beyond 256 take a kernel of their own with one column a
-// thread.  A request whose first row carries a negative position (a padding row of a captured step) is
-// skipped: its state slot belongs to someone else.
+// sequential in the tokens of its request.  A thread holds a tile of the state in registers, two
+// neighbouring rows (four beyond 128 rows) of four neighbouring columns, so that what it reads of q, b
+// and a serves four columns; rows go through the multipliers in pairs.  Eight lanes cover 16 (32) rows, and
+// so many groups of warps as are needed cover the rest.  Eight tokens' partial outputs are added over
+// the eight lanes together, each exchange halving the values a lane still holds; the groups' results meet in
+// shared memory and leave one round later.  Tokens are staged through shared memory in rounds: for
+// portions of prompts a first, fully parallel kernel writes q_t, b_t (and a_t) of every token as floats
+// (STEP_DECAY streams its rows as they are), and the recurrence streams them in with cp.async, two rounds
+// ahead of the one that is computed; single tokens are transformed as they are staged, in one kernel.
+// State rows beyond 256 take a kernel of their own with one column a thread.  A request whose first row
+// carries a negative position (a padding row of a captured step) is skipped: its state slot belongs to
+// someone else.
 #include <type_traits>
 
 #include "common.cuh"
@@ -395,9 +395,8 @@ __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
 }
 
 // The kernel for up to 256 state rows.  SLICES lanes, PAIRS pairs of rows a lane and PARTS groups of warps cover
-// the state's rows (padded); with two groups every output is the sum of two warps' results, which meet in
-// shared memory and leave for the result one round later.
-constexpr int TILE_WARPS = 8, TILE_THREADS = 32 * TILE_WARPS, TILE_STAGES = 4, BATCH = 8;
+// the state's rows (padded); every output is the sum of the groups' results, which meet in shared memory.
+constexpr int TILE_WARPS = 8, TILE_THREADS = 32 * TILE_WARPS, TILE_STAGES = 3, BATCH = 8;
 
 template <int SLICES, int PAIRS, int PARTS, int KIND>
 struct Tile {
@@ -408,7 +407,7 @@ struct Tile {
   static constexpr int cols = TILE_WARPS / PARTS * (32 / SLICES) * 4;        // value columns of a block
   static constexpr int round = rows <= 128 ? 16 : 8;                         // tokens staged together
   static constexpr int stage = planes * round * rows + round * cols + (per_token ? 2 * round : 0);
-  static constexpr int meet = PARTS == 1 ? 0 : 2 * PARTS * round * cols;     // results of two rounds
+  static constexpr int meet = 2 * PARTS * round * cols;                      // the groups' results of two rounds
   static constexpr size_t smem(int stages) { return sizeof(float) * (stages * stage + meet); }
 };
 
@@ -525,7 +524,7 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
     const float* vs = buf + planes * R * DP + cg * 4;
     const float* steps = buf + planes * R * DP + R * C;
     const float* qs = buf + row0;
-    float* mine = meet + ((turn2 * PARTS + part) * R) * C + cg * 4;  // (two groups of warps only)
+    float* mine = meet + ((turn2 * PARTS + part) * R) * C + cg * 4;
 #pragma unroll
     for (int r0 = 0; r0 < R; r0 += BATCH) {
       if (r0 >= n) break;
@@ -569,8 +568,8 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
 #pragma unroll
         for (int c = 0; c < 4; ++c) acc[k * 4 + c] = o[c];
       }
-      // sums over the slices: each exchange leaves a lane half of its values; lane `slice` ends with values
-      // slice * PER .. + PER - 1 of the BATCH * 4 (value k * 4 + c: token k, column c)
+      // sums over the slices: each exchange leaves a lane half of its values (value k * 4 + c: token k, column
+      // c), and lane `slice` ends with the four columns of token `slice`
       constexpr int PER = BATCH * 4 / SLICES;
 #pragma unroll
       for (int o = SLICES / 2, m = BATCH * 2; o > 0; o >>= 1, m >>= 1) {
@@ -582,17 +581,15 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
             acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
           }
       }
-#pragma unroll
-      for (int i = 0; i < PER; ++i) {
-        const int at = slice * PER + i, r = r0 + (at >> 2), c = at & 3;
-        if ((whole_round || r < n) && col0 + c < p.vdim) {
-          float y = acc[i];
-          if (per_token && part == 0) y = fmaf(skip, vs[r * C + c], y);
-          if (PARTS > 1)
-            mine[r * C + c] = y;
-          else
-            p.out[(size_t)(base + r) * p.ldo + (size_t)head * p.vdim + col0 + c] = y;
+      static_assert(PER == 4, "a lane ends with the four columns of one token");
+      const int r = r0 + slice;
+      if (whole_round || r < n) {
+        float4 y = make_float4(acc[0], acc[1], acc[2], acc[3]);
+        if (per_token && part == 0) {
+          const float4 v = *reinterpret_cast<const float4*>(vs + r * C);
+          y = make_float4(fmaf(skip, v.x, y.x), fmaf(skip, v.y, y.y), fmaf(skip, v.z, y.z), fmaf(skip, v.w, y.w));
         }
+        *reinterpret_cast<float4*>(mine + r * C) = y;
       }
     }
   };
@@ -605,18 +602,16 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
       compute_round(std::false_type{}, base, buf);
   };
 
-  // the results of the round at `base` that two groups of warps left (called behind a barrier)
+  // the outputs of the round at `base`, from what the groups of warps left (called behind a barrier)
   auto flush = [&](int base) {
-    if constexpr (PARTS > 1) {
-      const int n = min(R, t1 - base);
-      const float* r0 = meet + turn2 * PARTS * R * C;
-      for (int idx = tid; idx < n * C; idx += TILE_THREADS) {
-        const int c = blockIdx.x * C + idx % C;
-        float y = r0[idx];
+    const int n = min(R, t1 - base);
+    const float* r0 = meet + turn2 * PARTS * R * C;
+    for (int idx = tid; idx < n * C; idx += TILE_THREADS) {
+      const int c = blockIdx.x * C + idx % C;
+      float y = r0[idx];
 #pragma unroll
-        for (int k = 1; k < PARTS; ++k) y += r0[k * R * C + idx];
-        if (c < p.vdim) p.out[(size_t)(base + idx / C) * p.ldo + (size_t)head * p.vdim + c] = y;
-      }
+      for (int k = 1; k < PARTS; ++k) y += r0[k * R * C + idx];
+      if (c < p.vdim) p.out[(size_t)(base + idx / C) * p.ldo + (size_t)head * p.vdim + c] = y;
     }
   };
 
@@ -668,10 +663,8 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
       compute(base, tile_smem);
     }
   }
-  if (PARTS > 1) {
-    __syncthreads();
-    flush(t0 + (t1 - t0 - 1) / R * R);
-  }
+  __syncthreads();
+  flush(t0 + (t1 - t0 - 1) / R * R);
 #pragma unroll
   for (int k = 0; k < PAIRS; ++k) {
     float s[2][4];
@@ -702,8 +695,9 @@ int launch_tile_kind(const RecurrenceArgs& a, int S, cudaStream_t stream) {
                                   (int)L::smem(TILE_STAGES)));
     configured = true;
   }
-  recurrence_tile_kernel<SLICES, PAIRS, PARTS, KIND><<<dim3((a.vdim + L::cols - 1) / L::cols, a.H, S), TILE_THREADS,
-                                                       L::smem(a.streamed ? TILE_STAGES : 1), stream>>>(a);
+  const dim3 grid((a.vdim + L::cols - 1) / L::cols, a.H, S);
+  const size_t smem = L::smem(a.streamed ? TILE_STAGES : 1);
+  recurrence_tile_kernel<SLICES, PAIRS, PARTS, KIND><<<grid, TILE_THREADS, smem, stream>>>(a);
   DSP_CHECK_LAUNCH("dsp_linear_recurrence");
   return 0;
 }
@@ -801,10 +795,10 @@ extern "C" int dsp_linear_recurrence(const void* proj, int proj_dtype, long ld, 
     recurrence_prepare_kernel<<<(unsigned)(want < cap ? want : cap), 256, 0, stream>>>(a, T);
     DSP_CHECK_LAUNCH("dsp_linear_recurrence (first kernel)");
   }
-  if (dim <= 32) return launch_tile<16, 1, 1>(a, S, stream);
-  if (dim <= 64) return launch_tile<32, 1, 1>(a, S, stream);
-  if (dim <= 128) return launch_tile<32, 1, 2>(a, S, stream);
-  if (tiled) return launch_tile<32, 2, 2>(a, S, stream);
+  if (dim <= 32) return launch_tile<8, 1, 2>(a, S, stream);
+  if (dim <= 64) return launch_tile<8, 1, 4>(a, S, stream);
+  if (dim <= 128) return launch_tile<8, 1, 8>(a, S, stream);
+  if (tiled) return launch_tile<8, 2, 8>(a, S, stream);
   if (R == 16) return launch<16, 8>(a, S, smem, stream);
   return launch<32, 8>(a, S, smem, stream);
 }
