@@ -21,16 +21,17 @@
 //                 token and head and the value scaled by another (`steps`); o_t gets skip[head] * v_t on top:
 //                     S_t = a S_(t-1) + step b_t v_t^T,   o_t = S_t^T q_t + skip v_t
 //
-// One block of eight warps per (request, head, tile of value columns); what a block computes is
-// sequential in the tokens of its request.  A thread holds a tile of the state in registers, two
-// neighbouring rows (four beyond 128 rows) of four neighbouring columns, so that what it reads of q, b
-// and a serves four columns; rows go through the multipliers in pairs.  Eight lanes cover 16 (32) rows, and
-// so many groups of warps as are needed cover the rest.  Eight tokens' partial outputs are added over
-// the eight lanes together, each exchange halving the values a lane still holds; the groups' results meet in
-// shared memory and leave one round later.  Tokens are staged through shared memory in rounds: for
-// portions of prompts a first, fully parallel kernel writes q_t, b_t (and a_t) of every token as floats
+// One block per (request, head, tile of value columns); what a block computes is sequential in the
+// tokens of its request.  A thread holds a tile of the state in registers, a few neighbouring rows of four
+// neighbouring columns, so that what it reads of q, b and a serves four columns; rows go through the
+// multipliers in pairs.  Eight tokens' partial outputs are added over the lanes that share columns together,
+// each exchange halving the values a lane still holds.  Tokens are staged through shared memory in rounds.
+// Portions of prompts: a first, fully parallel kernel writes q_t, b_t (and a_t) of every token as floats
 // (STEP_DECAY streams its rows as they are), and the recurrence streams them in with cp.async, two rounds
-// ahead of the one that is computed; single tokens are transformed as they are staged, in one kernel.
+// ahead of the one that is computed; eight lanes cover 16 (32) state rows and groups of warps the rest (a lone
+// prompt leaves an SM one block: eight warps hide one another's latencies), the groups' results meet in
+// shared memory and leave one round later.  Single tokens: transformed as they are staged, in one kernel,
+// the lanes of a warp cover all the rows.
 // State rows beyond 256 take a kernel of their own with one column a thread.  A request whose first row
 // carries a negative position (a padding row of a captured step) is skipped: its state slot belongs to
 // someone else.
@@ -64,7 +65,6 @@ struct RecurrenceArgs {
   const float* steps;      // [T, 2, H]           STEP_DECAY: factor on the value, decay
   const float* skip;       // [H]                 STEP_DECAY
   int heads_per_group;     //                     STEP_DECAY (1 otherwise)
-  int streamed;            // rounds arrive by cp.async ahead of the computation (tile kernel)
   float* state;            // [slots, H, dim, vdim]
   const int* state_slot;   // [S]
   const int* q_start;      // [S + 1]
@@ -396,25 +396,26 @@ __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
 
 // The kernel for up to 256 state rows.  SLICES lanes, PAIRS pairs of rows a lane and PARTS groups of warps cover
 // the state's rows (padded); every output is the sum of the groups' results, which meet in shared memory.
-constexpr int TILE_WARPS = 8, TILE_THREADS = 32 * TILE_WARPS, TILE_STAGES = 3, BATCH = 8;
+constexpr int TILE_STAGES = 3, BATCH = 8;
 
-template <int SLICES, int PAIRS, int PARTS, int KIND>
+template <int SLICES, int PAIRS, int PARTS, int WARPS, bool STREAMED, int KIND>
 struct Tile {
   static constexpr bool gate = KIND == VECTOR_DECAY, per_token = KIND == TOKEN_DECAY;
   static constexpr int planes = gate ? 3 : 2;
   static constexpr int part_rows = SLICES * 2 * PAIRS;                       // state rows of a group of warps
   static constexpr int rows = part_rows * PARTS;                             // state rows, padded
-  static constexpr int cols = TILE_WARPS / PARTS * (32 / SLICES) * 4;        // value columns of a block
+  static constexpr int cols = WARPS / PARTS * (32 / SLICES) * 4;             // value columns of a block
   static constexpr int round = rows <= 128 ? 16 : 8;                         // tokens staged together
   static constexpr int stage = planes * round * rows + round * cols + (per_token ? 2 * round : 0);
-  static constexpr int meet = 2 * PARTS * round * cols;                      // the groups' results of two rounds
-  static constexpr size_t smem(int stages) { return sizeof(float) * (stages * stage + meet); }
+  static constexpr int meet = PARTS == 1 ? 0 : 2 * PARTS * round * cols;     // the groups' results of two rounds
+  static constexpr int stages = STREAMED ? TILE_STAGES : 1;
+  static constexpr size_t smem = sizeof(float) * (stages * stage + meet);
 };
 
-template <int SLICES, int PAIRS, int PARTS, int KIND>
-__global__ void __launch_bounds__(TILE_THREADS, 2)
+template <int SLICES, int PAIRS, int PARTS, int WARPS, bool STREAMED, int KIND>
+__global__ void __launch_bounds__(32 * WARPS, 2)
 recurrence_tile_kernel(const RecurrenceArgs p) {
-  using L = Tile<SLICES, PAIRS, PARTS, KIND>;
+  using L = Tile<SLICES, PAIRS, PARTS, WARPS, STREAMED, KIND>;
   constexpr bool gate = L::gate, per_token = L::per_token;
   constexpr int DP = L::rows, C = L::cols, R = L::round, planes = L::planes;
   extern __shared__ __align__(16) float tile_smem[];
@@ -422,11 +423,10 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
   const int t0 = p.q_start[seq], t1 = p.q_start[seq + 1];
   if (t1 <= t0 || p.positions[t0] < 0) return;
   const int tid = threadIdx.x, lane = tid & 31, slice = lane % SLICES;
-  constexpr int PART_WARPS = TILE_WARPS / PARTS;
+  constexpr int TILE_THREADS = 32 * WARPS, PART_WARPS = WARPS / PARTS;
   const int part = (tid >> 5) / PART_WARPS;  // this warp's group of state rows
   const int cg = (tid >> 5) % PART_WARPS * (32 / SLICES) + lane / SLICES;  // this thread's group of four columns
   const int col0 = blockIdx.x * C + cg * 4;
-  const bool streamed = p.streamed != 0;
   const float* rows = reinterpret_cast<const float*>(p.proj);
   const bool whole = p.ld % 4 == 0 && (((uintptr_t)rows) & 15) == 0;
   const bool wide = p.dim % 4 == 0 && (per_token ? whole && p.q_off % 4 == 0 && p.k_off % 4 == 0 : (((uintptr_t)p.ready) & 15) == 0);
@@ -464,7 +464,7 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
 
   // rows and columns beyond the head's own stay zero in every stage: written here and never again
   if (DP > p.dim || (int)(blockIdx.x + 1) * C > p.vdim) {
-    for (int idx = tid; idx < (streamed ? TILE_STAGES : 1) * L::stage; idx += TILE_THREADS) tile_smem[idx] = 0.f;
+    for (int idx = tid; idx < L::stages * L::stage; idx += TILE_THREADS) tile_smem[idx] = 0.f;
     __syncthreads();
   }
 
@@ -515,7 +515,7 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
       cp_async4(vs + R * C + (tid & 1) * R + (tid >> 1), p.steps + ((size_t)(base + (tid >> 1)) * 2 + (tid & 1)) * p.H + head);
   };
 
-  float* meet = tile_smem + (streamed ? TILE_STAGES : 1) * L::stage;
+  float* meet = tile_smem + L::stages * L::stage;
   int turn2 = 0;  // which of the two meeting places the latest round used
   // one round; `full`: all of its tokens are there (no conditions between the tokens' loads)
   auto compute_round = [&](auto full, int base, const float* buf) {
@@ -568,8 +568,8 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
 #pragma unroll
         for (int c = 0; c < 4; ++c) acc[k * 4 + c] = o[c];
       }
-      // sums over the slices: each exchange leaves a lane half of its values (value k * 4 + c: token k, column
-      // c), and lane `slice` ends with the four columns of token `slice`
+      // sums over the slices: each exchange leaves a lane half of its values, and lane `slice` ends with values
+      // slice * PER .. + PER - 1 of the BATCH * 4 (value k * 4 + c: token k, column c)
       constexpr int PER = BATCH * 4 / SLICES;
 #pragma unroll
       for (int o = SLICES / 2, m = BATCH * 2; o > 0; o >>= 1, m >>= 1) {
@@ -581,15 +581,18 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
             acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
           }
       }
-      static_assert(PER == 4, "a lane ends with the four columns of one token");
-      const int r = r0 + slice;
-      if (whole_round || r < n) {
-        float4 y = make_float4(acc[0], acc[1], acc[2], acc[3]);
-        if (per_token && part == 0) {
-          const float4 v = *reinterpret_cast<const float4*>(vs + r * C);
-          y = make_float4(fmaf(skip, v.x, y.x), fmaf(skip, v.y, y.y), fmaf(skip, v.z, y.z), fmaf(skip, v.w, y.w));
+#pragma unroll
+      for (int i = 0; i < PER; ++i) {
+        const int at = slice * PER + i, r = r0 + (at >> 2), c = at & 3;
+        if (whole_round || r < n) {
+          if (per_token && part == 0) acc[i] = fmaf(skip, vs[r * C + c], acc[i]);
+          if (PARTS == 1 && col0 + c < p.vdim) p.out[(size_t)(base + r) * p.ldo + (size_t)head * p.vdim + col0 + c] = acc[i];
         }
-        *reinterpret_cast<float4*>(mine + r * C) = y;
+      }
+      if constexpr (PARTS > 1) {
+        static_assert(PER == 4, "a lane ends with the four columns of one token");
+        if (whole_round || r0 + slice < n)
+          *reinterpret_cast<float4*>(mine + (r0 + slice) * C) = make_float4(acc[0], acc[1], acc[2], acc[3]);
       }
     }
   };
@@ -604,18 +607,20 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
 
   // the outputs of the round at `base`, from what the groups of warps left (called behind a barrier)
   auto flush = [&](int base) {
-    const int n = min(R, t1 - base);
-    const float* r0 = meet + turn2 * PARTS * R * C;
-    for (int idx = tid; idx < n * C; idx += TILE_THREADS) {
-      const int c = blockIdx.x * C + idx % C;
-      float y = r0[idx];
+    if constexpr (PARTS > 1) {
+      const int n = min(R, t1 - base);
+      const float* r0 = meet + turn2 * PARTS * R * C;
+      for (int idx = tid; idx < n * C; idx += TILE_THREADS) {
+        const int c = blockIdx.x * C + idx % C;
+        float y = r0[idx];
 #pragma unroll
-      for (int k = 1; k < PARTS; ++k) y += r0[k * R * C + idx];
-      if (c < p.vdim) p.out[(size_t)(base + idx / C) * p.ldo + (size_t)head * p.vdim + c] = y;
+        for (int k = 1; k < PARTS; ++k) y += r0[k * R * C + idx];
+        if (c < p.vdim) p.out[(size_t)(base + idx / C) * p.ldo + (size_t)head * p.vdim + c] = y;
+      }
     }
   };
 
-  if (streamed) {
+  if constexpr (STREAMED) {
     for (int s = 0; s < TILE_STAGES - 1; ++s) {
       if (t0 + s * R < t1) stage_round(t0 + s * R, tile_smem + s * L::stage);
       asm volatile("cp.async.commit_group;\n");
@@ -663,8 +668,10 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
       compute(base, tile_smem);
     }
   }
-  __syncthreads();
-  flush(t0 + (t1 - t0 - 1) / R * R);
+  if constexpr (PARTS > 1) {
+    __syncthreads();
+    flush(t0 + (t1 - t0 - 1) / R * R);
+  }
 #pragma unroll
   for (int k = 0; k < PAIRS; ++k) {
     float s[2][4];
@@ -686,27 +693,26 @@ recurrence_tile_kernel(const RecurrenceArgs p) {
   }
 }
 
-template <int SLICES, int PAIRS, int PARTS, int KIND>
+template <int SLICES, int PAIRS, int PARTS, int WARPS, bool STREAMED, int KIND>
 int launch_tile_kind(const RecurrenceArgs& a, int S, cudaStream_t stream) {
-  using L = Tile<SLICES, PAIRS, PARTS, KIND>;
+  using L = Tile<SLICES, PAIRS, PARTS, WARPS, STREAMED, KIND>;
   static bool configured = false;
   if (!configured) {
-    DSP_CUDA(cudaFuncSetAttribute(recurrence_tile_kernel<SLICES, PAIRS, PARTS, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                  (int)L::smem(TILE_STAGES)));
+    DSP_CUDA(cudaFuncSetAttribute(recurrence_tile_kernel<SLICES, PAIRS, PARTS, WARPS, STREAMED, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                  (int)L::smem));
     configured = true;
   }
   const dim3 grid((a.vdim + L::cols - 1) / L::cols, a.H, S);
-  const size_t smem = L::smem(a.streamed ? TILE_STAGES : 1);
-  recurrence_tile_kernel<SLICES, PAIRS, PARTS, KIND><<<grid, TILE_THREADS, smem, stream>>>(a);
+  recurrence_tile_kernel<SLICES, PAIRS, PARTS, WARPS, STREAMED, KIND><<<grid, 32 * WARPS, L::smem, stream>>>(a);
   DSP_CHECK_LAUNCH("dsp_linear_recurrence");
   return 0;
 }
 
-template <int SLICES, int PAIRS, int PARTS>
+template <int SLICES, int PAIRS, int PARTS, int WARPS, bool STREAMED>
 int launch_tile(const RecurrenceArgs& a, int S, cudaStream_t stream) {
-  if (a.mode == STEP_DECAY) return launch_tile_kind<SLICES, PAIRS, PARTS, TOKEN_DECAY>(a, S, stream);
-  if (a.mode == FIXED_DECAY) return launch_tile_kind<SLICES, PAIRS, PARTS, SCALAR_DECAY>(a, S, stream);
-  return launch_tile_kind<SLICES, PAIRS, PARTS, VECTOR_DECAY>(a, S, stream);
+  if (a.mode == STEP_DECAY) return launch_tile_kind<SLICES, PAIRS, PARTS, WARPS, STREAMED, TOKEN_DECAY>(a, S, stream);
+  if (a.mode == FIXED_DECAY) return launch_tile_kind<SLICES, PAIRS, PARTS, WARPS, STREAMED, SCALAR_DECAY>(a, S, stream);
+  return launch_tile_kind<SLICES, PAIRS, PARTS, WARPS, STREAMED, VECTOR_DECAY>(a, S, stream);
 }
 
 template <int ROWS, int TPR, int KIND>
@@ -769,7 +775,6 @@ extern "C" int dsp_linear_recurrence(const void* proj, int proj_dtype, long ld, 
   a.steps = steps; a.skip = skip; a.heads_per_group = mode == STEP_DECAY ? heads_per_group : 1;
   a.state = state; a.state_slot = state_slot; a.q_start = q_start; a.positions = positions;
   a.out = out; a.ldo = ldo; a.ready = scratch;
-  a.streamed = scratch != nullptr || (mode == STEP_DECAY && T > 2 * S);
   // one column a thread, 32 threads a column, 16 or 32 state rows a thread (beyond 256 state rows)
   const bool tiled = dim <= 256;
   const int slices = 32, rows = (dim + slices - 1) / slices;
@@ -795,10 +800,17 @@ extern "C" int dsp_linear_recurrence(const void* proj, int proj_dtype, long ld, 
     recurrence_prepare_kernel<<<(unsigned)(want < cap ? want : cap), 256, 0, stream>>>(a, T);
     DSP_CHECK_LAUNCH("dsp_linear_recurrence (first kernel)");
   }
-  if (dim <= 32) return launch_tile<8, 1, 2>(a, S, stream);
-  if (dim <= 64) return launch_tile<8, 1, 4>(a, S, stream);
-  if (dim <= 128) return launch_tile<8, 1, 8>(a, S, stream);
-  if (tiled) return launch_tile<8, 2, 8>(a, S, stream);
+  if (scratch || (mode == STEP_DECAY && T > 2 * S)) {  // portions of prompts
+    if (dim <= 32) return launch_tile<8, 1, 2, 8, true>(a, S, stream);
+    if (dim <= 64) return launch_tile<8, 1, 4, 8, true>(a, S, stream);
+    if (dim <= 128) return launch_tile<8, 1, 8, 8, true>(a, S, stream);
+    if (tiled) return launch_tile<8, 2, 8, 8, true>(a, S, stream);
+  } else {  // single tokens
+    if (dim <= 32) return launch_tile<8, 2, 1, 4, false>(a, S, stream);
+    if (dim <= 64) return launch_tile<16, 2, 1, 4, false>(a, S, stream);
+    if (dim <= 128) return launch_tile<32, 2, 1, 4, false>(a, S, stream);
+    if (tiled) return launch_tile<32, 4, 1, 4, false>(a, S, stream);
+  }
   if (R == 16) return launch<16, 8>(a, S, smem, stream);
   return launch<32, 8>(a, S, smem, stream);
 }
