@@ -84,10 +84,37 @@ __device__ __forceinline__ float4 conv_at4(const ConvIn& p, const float* row, in
   }
   return acc;
 }
-// whether conv_at4 serves token i: not one of those whose taps reach into the state slot
-__device__ __forceinline__ bool in_fours(const ConvIn& p, int i) {
-  return p.w && p.dtype == DSP_F32 && i >= p.taps - 1 && p.channels % 4 == 0 && p.off % 4 == 0 && p.ld % 4 == 0 &&
-         (((uintptr_t)p.u | (uintptr_t)p.w) & 15) == 0;
+// whether rows, weights and slots can be taken four channels at a time
+__device__ __forceinline__ bool in_fours(const ConvIn& p) {
+  return p.w && p.dtype == DSP_F32 && p.channels % 4 == 0 && p.off % 4 == 0 && p.ld % 4 == 0 &&
+         (((uintptr_t)p.u | (uintptr_t)p.w | (uintptr_t)p.hist) & 15) == 0;
+}
+
+// A portion of one token (decoding): four neighbouring channels' convolution and the new state in one
+// pass, every load issued before the first value is used.  The same sums in the same order.
+constexpr int SINGLE_TAPS = 8;
+__device__ __forceinline__ bool is_single(const ConvIn& p, const Turn& r) {
+  return r.n == 1 && p.taps > 1 && p.taps <= SINGLE_TAPS && in_fours(p);
+}
+__device__ __forceinline__ float4 conv_single4(const ConvIn& p, const float* row, float* hist, int c) {
+  float4 x[SINGLE_TAPS], acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int j = 0; j < SINGLE_TAPS; ++j)
+    if (j < p.taps)
+      x[j] = *reinterpret_cast<const float4*>(j < p.taps - 1 ? hist + (size_t)j * p.channels + c : row + p.off + c);
+#pragma unroll
+  for (int j = 0; j < SINGLE_TAPS; ++j)
+    if (j < p.taps) {
+      const float4 w = *reinterpret_cast<const float4*>(p.w + (size_t)j * p.channels + c);
+      acc.x = fmaf(w.x, x[j].x, acc.x);
+      acc.y = fmaf(w.y, x[j].y, acc.y);
+      acc.z = fmaf(w.z, x[j].z, acc.z);
+      acc.w = fmaf(w.w, x[j].w, acc.w);
+    }
+#pragma unroll
+  for (int j = 1; j < SINGLE_TAPS; ++j)
+    if (j < p.taps) *reinterpret_cast<float4*>(hist + (size_t)(j - 1) * p.channels + c) = x[j];
+  return acc;
 }
 
 // leaves the portion's last taps - 1 inputs of channel c in the slot (in place: row m is written before
@@ -110,10 +137,12 @@ conv_steps_kernel(const ConvIn p, const float* __restrict__ bias, float* __restr
   const Turn r = turn_of(p, t);
   float* hist = p.hist + (size_t)p.state_slot[r.seq] * (p.taps - 1) * p.channels;
   auto silu = [](float v) { return v / (1.f + expf(-v)); };
-  if (!r.owner && r.count == 1 && in_fours(p, r.first) && ldo % 4 == 0 && ((uintptr_t)out & 15) == 0 && ((uintptr_t)bias & 15) == 0) {
+  const bool single = is_single(p, r);
+  if ((single || (!r.owner && r.count == 1 && in_fours(p))) && ldo % 4 == 0 && ((uintptr_t)out & 15) == 0 && ((uintptr_t)bias & 15) == 0) {
     const int c = (blockIdx.y * 256 + threadIdx.x) * 4;
     if (c < p.channels) {
-      float4 v = conv_at4(p, reinterpret_cast<const float*>(p.u) + (size_t)t * p.ld, c);
+      const float* row = reinterpret_cast<const float*>(p.u) + (size_t)t * p.ld;
+      float4 v = single ? conv_single4(p, row, hist, c) : conv_at4(p, row, c);
       if (bias) {
         const float4 b = *reinterpret_cast<const float4*>(bias + c);
         v.x += b.x, v.y += b.y, v.z += b.z, v.w += b.w;
@@ -128,12 +157,12 @@ conv_steps_kernel(const ConvIn p, const float* __restrict__ bias, float* __restr
         if (c >= p.channels) break;
         out[(size_t)(r.row0 + i) * ldo + c] = silu(conv_at(p, r, hist, c, i) + (bias ? bias[c] : 0.f));
       }
+    if (r.owner)
+      for (int k = 0; k < PER_THREAD; ++k) {
+        const int c = (blockIdx.y * PER_THREAD + k) * 256 + threadIdx.x;
+        if (c < p.channels) keep_inputs(p, r, hist, c);
+      }
   }
-  if (r.owner)
-    for (int k = 0; k < PER_THREAD; ++k) {
-      const int c = (blockIdx.y * PER_THREAD + k) * 256 + threadIdx.x;
-      if (c < p.channels) keep_inputs(p, r, hist, c);
-    }
   if (blockIdx.y == 0)
     for (int h = threadIdx.x; h < heads; h += blockDim.x) {
       const float step = softplus_f(ld_any(p.u, p.dtype, (size_t)t * p.ld + step_off + h) + step_bias[h]);
@@ -154,13 +183,15 @@ qkv_conv_rotate_store_kernel(const ConvIn p, const int* __restrict__ page_table,
   if (r.count == 0) return;
   float* hist = p.taps > 1 ? p.hist + (size_t)p.state_slot[r.seq] * (p.taps - 1) * p.channels : nullptr;
   float* cs = row + p.channels;
+  const bool single = is_single(p, r);
   const int half = rot / 2, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
   for (int i = r.first; i < r.first + r.count; ++i) {
     const int tok = r.row0 + i, pos = p.positions[tok];
-    if (in_fours(p, i))
+    if (single || (in_fours(p) && i >= p.taps - 1)) {
+      const float* u = reinterpret_cast<const float*>(p.u) + (size_t)tok * p.ld;
       for (int c = tid * 4; c < p.channels; c += blockDim.x * 4)
-        *reinterpret_cast<float4*>(row + c) = conv_at4(p, reinterpret_cast<const float*>(p.u) + (size_t)tok * p.ld, c);
-    else
+        *reinterpret_cast<float4*>(row + c) = single ? conv_single4(p, u, hist, c) : conv_at4(p, u, c);
+    } else
       for (int c = tid; c < p.channels; c += blockDim.x) row[c] = conv_at(p, r, hist, c, i);
     for (int m = tid; m < half; m += blockDim.x) sincosf((float)pos * inv_freq[m], &cs[half + m], &cs[m]);
     __syncthreads();
@@ -196,7 +227,7 @@ qkv_conv_rotate_store_kernel(const ConvIn p, const int* __restrict__ page_table,
     }
     __syncthreads();  // the row is taken again
   }
-  if (r.owner && p.taps > 1)
+  if (r.owner && p.taps > 1 && !single)
     for (int c = tid; c < p.channels; c += blockDim.x) keep_inputs(p, r, hist, c);
 }
 
