@@ -21,6 +21,8 @@
 // stretches: both the query's and the key's part are, so their product carries mag^2).
 // `window` W > 0: the query at position p sees the keys j with p - W < j <= p (0: every j <= p);
 // older keys are never looked up, their pages may have been given back.
+// `sink` (float [H]): the softmax has one more key of score sink[h] (unscaled) and no value: the running
+// pair of the online softmax starts at (max, sum) = (sink[h], 1) instead of (-inf, 0).
 //
 // pools: latent [num_pages, 1, page_size, R], rotated key [num_pages, 1, page_size, r];
 // page = page_table[seq * pt_stride + position / page_size].
@@ -105,7 +107,7 @@ attn_latent_kernel(const float* __restrict__ qa, long ldqa, const void* __restri
                    int layout, float mag, int window, const T* __restrict__ c_pool, const T* __restrict__ r_pool,
                    const int* __restrict__ page_table, int pt_stride, const int* __restrict__ positions,
                    const int* __restrict__ seq_of_token, void* __restrict__ out, int out_dtype, long ldo,
-                   int H, int R, int r, int page_size, int num_pages, float scale, int* err) {
+                   int H, int R, int r, int page_size, int num_pages, float scale, const float* __restrict__ sink, int* err) {
   extern __shared__ float smem[];
   const int W = R + r;
   float* qs = smem;                        // [GCHUNK][W]
@@ -143,8 +145,8 @@ attn_latent_kernel(const float* __restrict__ qa, long ldqa, const void* __restri
   float m[GCHUNK], l[GCHUNK], acc[GCHUNK][DPT];
 #pragma unroll
   for (int g = 0; g < GCHUNK; ++g) {
-    m[g] = -INFINITY;
-    l[g] = 0.f;
+    m[g] = sink && g < gn ? sink[h0 + g] : -INFINITY;
+    l[g] = sink ? 1.f : 0.f;
 #pragma unroll
     for (int j = 0; j < DPT; ++j) acc[g][j] = 0.f;
   }
@@ -250,7 +252,7 @@ int launch_attn(const float* qa, long ldqa, const void* q, int q_dtype, long ldq
                 int qr_off, const float* inv_freq, int rot, int layout, float mag, int window, const void* c_pool,
                 const void* r_pool, const int* page_table, int pt_stride, const int* positions, const int* seq_of_token,
                 void* out, int out_dtype, long ldo, int T_, int H, int R, int r, int page_size,
-                int num_pages, float scale, int* err, cudaStream_t stream) {
+                int num_pages, float scale, const float* sink, int* err, cudaStream_t stream) {
   const size_t smem = (size_t)(GCHUNK * (R + r) + GCHUNK * THREADS) * sizeof(float) + THREADS * sizeof(long);
   static size_t configured = 48 * 1024;
   if (smem > configured) {
@@ -261,7 +263,7 @@ int launch_attn(const float* qa, long ldqa, const void* q, int q_dtype, long ldq
   DSP_CUDA(launch_plain(attn_latent_kernel<T, DPT>, grid, dim3(THREADS), smem, stream, qa, ldqa, q, q_dtype,
                       ldq, q_head_stride, qr_off, inv_freq, rot, layout, mag, window, (const T*)c_pool, (const T*)r_pool,
                       page_table, pt_stride, positions, seq_of_token, out, out_dtype, ldo, H, R, r,
-                      page_size, num_pages, scale, err));
+                      page_size, num_pages, scale, sink, err));
   DSP_CHECK_LAUNCH("dsp_attn_latent");
   return 0;
 }
@@ -293,7 +295,7 @@ extern "C" int dsp_attn_latent(const float* qa, long ldqa, const void* q, int q_
                                float mag, int window, const void* c_pool, const void* r_pool, int pool_dtype,
                                const int* page_table, int pt_stride, const int* positions,
                                const int* seq_of_token, void* out, int out_dtype, long ldo, int T_, int H,
-                               int R, int r, int page_size, int num_pages, float scale,
+                               int R, int r, int page_size, int num_pages, float scale, const float* sink,
                                cudaStream_t stream) {
   if (T_ == 0) return 0;
   int* err = dsp_device_error_ptr();
@@ -305,7 +307,7 @@ extern "C" int dsp_attn_latent(const float* qa, long ldqa, const void* q, int q_
   DSP_REQUIRE((layout == 0 || layout == 1) && window >= 0, "dsp_attn_latent: layout=%d window=%d", layout, window);
 #define DSP_LATENT_ARGS qa, ldqa, q, q_dtype, ldq, q_head_stride, qr_off, inv_freq, rot, layout, mag, window, c_pool, r_pool, page_table, \
                         pt_stride, positions, seq_of_token, out, out_dtype, ldo, T_, H, R, r, page_size, num_pages,  \
-                        scale, err, stream
+                        scale, sink, err, stream
   const int dpt = (R + THREADS - 1) / THREADS;
   if (pool_dtype == DSP_F32) {
     if (dpt <= 1) return launch_attn<float, 1>(DSP_LATENT_ARGS);
@@ -338,7 +340,9 @@ extern "C" int dsp_attn_latent(const float* qa, long ldqa, const void* q, int q_
 // The key tiles of a tile can be cut into `splits` ranges (grid.z), each leaving an unnormalised
 // partial and (maximum in the base-2 domain, sum) per row for dsp_attn_combine: single tokens
 // with long contexts then fill the device.  Keys beyond the tile's last position are never
-// loaded (zero rows); a page id outside the pool is recorded and its rows are zero.
+// loaded (zero rows); a page id outside the pool is recorded and its rows are zero.  The output
+// columns are padded to whole 64s (columns beyond R are computed from whatever follows the latent in
+// the key row and never stored).  The sink is counted by the first key range only.
 namespace tc {
 constexpr int BM = 64, BN = 32, THREADS = 512, P_ROWB = 80, S_ROW = BN + 4;
 
@@ -354,6 +358,7 @@ struct Args {
   float* part_o; float* part_ml; int splits;
   int H, HC, TPT, R, r, page_size, num_pages;
   float scale_log2;
+  const float* sink;
   int* err;
 };
 
@@ -384,13 +389,14 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
-__host__ __device__ inline int key_row_bytes(int W) { return ((W * 2 + 127) / 128) * 128 + 16; }
+// bytes of a key row in shared memory: the row itself, or the padded output columns where those are more
+__host__ __device__ inline int key_row_bytes(int W, int cols) { return (((W > cols ? W : cols) * 2 + 127) / 128) * 128 + 16; }
 
-// NT16: blocks of 16 output columns per warp = R / 64
+// NT16: blocks of 16 output columns per warp (R / 64, rounded up)
 template <int NT16>
 __global__ void __launch_bounds__(THREADS, 1) attn_latent_mma_kernel(const Args p) {
   extern __shared__ __align__(128) unsigned char smem[];
-  const int W = p.R + p.r, ROWB = key_row_bytes(W), CH = W / 8, CH_LAT = p.R / 8;
+  const int W = p.R + p.r, ROWB = key_row_bytes(W, NT16 * 64), CH = W / 8, CH_LAT = p.R / 8;
   const uint32_t q_s = (uint32_t)__cvta_generic_to_shared(smem);
   const uint32_t k_s = q_s + BM * ROWB;
   const uint32_t p_s = k_s + 2 * BN * ROWB;
@@ -502,6 +508,11 @@ __global__ void __launch_bounds__(THREADS, 1) attn_latent_mma_kernel(const Args 
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[i][e] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+  if (p.sink && blockIdx.z == 0) {  // in the base-2 domain of the scores
+    m_run[0] = p.sink[head0 + row_a % hc] * 1.4426950408889634f;
+    m_run[1] = p.sink[head0 + row_b % hc] * 1.4426950408889634f;
+    l_run[0] = l_run[1] = 1.f;
+  }
   const int pos_a = row_a < nrows ? pos0 + row_a / hc : -1, pos_b = row_b < nrows ? pos0 + row_b / hc : -1;
   const int reach = p.window > 0 ? p.window : 0x40000000;
 
@@ -629,12 +640,13 @@ __global__ void __launch_bounds__(THREADS, 1) attn_latent_mma_kernel(const Args 
       bf16* dst = p.out + (size_t)t * p.ldo + (size_t)hd * p.R + cg * NT16 * 16 + 2 * c4;
 #pragma unroll
       for (int i = 0; i < 2 * NT16; ++i)
-        *reinterpret_cast<uint32_t*>(dst + i * 8) = pack_bf16(o[i][2 * r] * inv, o[i][2 * r + 1] * inv);
+        if (cg * NT16 * 16 + i * 8 < p.R) *reinterpret_cast<uint32_t*>(dst + i * 8) = pack_bf16(o[i][2 * r] * inv, o[i][2 * r + 1] * inv);
     } else {
       const size_t row = (size_t)t * p.H + hd;
       float* dst = p.part_o + (row * p.splits + blockIdx.z) * p.R + cg * NT16 * 16 + 2 * c4;
 #pragma unroll
-      for (int i = 0; i < 2 * NT16; ++i) *reinterpret_cast<float2*>(dst + i * 8) = make_float2(o[i][2 * r], o[i][2 * r + 1]);
+      for (int i = 0; i < 2 * NT16; ++i)
+        if (cg * NT16 * 16 + i * 8 < p.R) *reinterpret_cast<float2*>(dst + i * 8) = make_float2(o[i][2 * r], o[i][2 * r + 1]);
       if (cg == 0 && c4 == 0) {
         p.part_ml[(row * p.splits + blockIdx.z) * 2] = m_run[r];
         p.part_ml[(row * p.splits + blockIdx.z) * 2 + 1] = l_run[r];
@@ -645,7 +657,7 @@ __global__ void __launch_bounds__(THREADS, 1) attn_latent_mma_kernel(const Args 
 
 template <int NT16>
 int launch(const Args& a, int num_tiles, int head_chunks, cudaStream_t stream) {
-  const int ROWB = key_row_bytes(a.R + a.r);
+  const int ROWB = key_row_bytes(a.R + a.r, NT16 * 64);
   const size_t smem = (size_t)BM * ROWB + 2 * (size_t)BN * ROWB + BM * P_ROWB + (2 * BM * 4 + 4 * BM * S_ROW) * sizeof(float);
   if (smem > 227 * 1024) return 2;
   static bool configured = false;
@@ -662,7 +674,7 @@ int launch(const Args& a, int num_tiles, int head_chunks, cudaStream_t stream) {
 
 // Tiles tile_offset .. tile_offset + num_tiles - 1 of the tile list (TPT tokens a tile).  splits > 1:
 // unnormalised partials go to part_o [rows, splits, R] and part_ml [rows, splits, 2], rows being
-// flat token * H + head.  Sizes: R a multiple of 64 up to 512 (not 320 or 448), r a multiple of 16,
+// flat token * H + head.  Sizes: R and r multiples of 16, R up to 512,
 // row strides of qa in pairs of floats, pools and out in bfloat16.
 extern "C" int dsp_attn_latent_mma(const float* qa, long ldqa, const void* q, int q_dtype, long ldq,
                                    int q_head_stride, int qr_off, const float* inv_freq, int rot, int layout,
@@ -671,11 +683,11 @@ extern "C" int dsp_attn_latent_mma(const float* qa, long ldqa, const void* q, in
                                    const int* tile_seq, const int* tile_tok0, int tile_offset,
                                    int num_tiles, void* out, long ldo, float* part_o, float* part_ml,
                                    int splits, int H, int TPT, int R, int r, int page_size, int num_pages,
-                                   float scale, cudaStream_t stream) {
+                                   float scale, const float* sink, cudaStream_t stream) {
   if (num_tiles == 0) return 0;
   int* err = dsp_device_error_ptr();
   DSP_REQUIRE(err != nullptr, "dsp_attn_latent_mma: no device error word");
-  DSP_REQUIRE(R % 64 == 0 && r % 16 == 0 && r >= 0 && rot % 2 == 0 && rot <= r, "dsp_attn_latent_mma: R=%d r=%d rot=%d", R, r, rot);
+  DSP_REQUIRE(R > 0 && R <= 512 && R % 16 == 0 && r % 16 == 0 && r >= 0 && rot % 2 == 0 && rot <= r, "dsp_attn_latent_mma: R=%d r=%d rot=%d", R, r, rot);
   DSP_REQUIRE((layout == 0 || layout == 1) && window >= 0, "dsp_attn_latent_mma: layout=%d window=%d", layout, window);
   DSP_REQUIRE(ldqa % 2 == 0 && ((uintptr_t)qa % 8) == 0 && ldo % 2 == 0 && ((uintptr_t)out % 4) == 0 &&
               ((uintptr_t)c_pool % 16) == 0 && ((uintptr_t)r_pool % 16) == 0, "dsp_attn_latent_mma: operand alignment");
@@ -690,15 +702,18 @@ extern "C" int dsp_attn_latent_mma(const float* qa, long ldqa, const void* q, in
   a.out = (bf16*)out; a.ldo = ldo; a.part_o = part_o; a.part_ml = part_ml; a.splits = splits;
   a.H = H; a.HC = HC; a.TPT = TPT; a.R = R; a.r = r; a.page_size = page_size; a.num_pages = num_pages;
   a.scale_log2 = scale * 1.4426950408889634f;
+  a.sink = sink;
   a.err = err;
   const int chunks = (H + HC - 1) / HC;
   int rc;
-  switch (R / 64) {
+  switch ((R + 63) / 64) {
     case 1: rc = tc::launch<1>(a, num_tiles, chunks, stream); break;
     case 2: rc = tc::launch<2>(a, num_tiles, chunks, stream); break;
     case 3: rc = tc::launch<3>(a, num_tiles, chunks, stream); break;
     case 4: rc = tc::launch<4>(a, num_tiles, chunks, stream); break;
+    case 5:
     case 6: rc = tc::launch<6>(a, num_tiles, chunks, stream); break;
+    case 7:
     case 8: rc = tc::launch<8>(a, num_tiles, chunks, stream); break;
     default: DSP_REQUIRE(false, "dsp_attn_latent_mma: latent size %d is not built", R);
   }

@@ -16,6 +16,8 @@
 //     position * v_inv_freq[m], after the norm (the attention kernel turns its result back by the
 //     query's position, so that a value enters the sum turned by the distance),
 //   * with `qt_every` > 0: multiplies every query by 1 + qt_coef * ln(floor((position + 1) / qt_every) + 1),
+//   * with `v_from_k`: has no value columns in the row; a token's values are its projected keys, as they are
+//     before norm and rotation (Dv = Dk),
 //   * writes the query to `q_out` [T, H * Dk] and the key and the value to the pages (pools
 //     [num_pages, G, page_size, Dk] and [.., Dv]) in the pools' type.
 // With `maps` = M > 1 every query and key head consists of M parts of Dk values that are normed and
@@ -41,7 +43,7 @@ qkv_rotate_store_kernel(const void* __restrict__ qkv, int in_dtype, long ld, con
                         void* __restrict__ k_pool, void* __restrict__ v_pool, int pool_dtype,
                         const float* __restrict__ inv_freq, int rot, const void* __restrict__ v_other, int vo_dtype,
                         long ld_vo, const float* __restrict__ lambda, const float* __restrict__ q_norm_w,
-                        const float* __restrict__ k_norm_w, float norm_eps, int v_norm,
+                        const float* __restrict__ k_norm_w, float norm_eps, int v_norm, int v_from_k,
                         const float* __restrict__ v_inv_freq, void* __restrict__ q_out, long ld_q, int H,
                         int G, int Dk, int Dv, int maps, float qt_coef, int qt_every, int page_size, int num_pages,
                         int write_kv, int* err) {
@@ -59,7 +61,7 @@ qkv_rotate_store_kernel(const void* __restrict__ qkv, int in_dtype, long ld, con
   const int G_v = G;
   H *= maps;  // from here on H and G count the parts of query and key heads
   G *= maps;
-  const size_t k0 = row + (size_t)H * Dk, v0 = k0 + (size_t)G * Dk;
+  const size_t k0 = row + (size_t)H * Dk, v0 = v_from_k ? k0 : k0 + (size_t)G * Dk;
   const float q_temp = qt_every > 0 ? 1.f + qt_coef * logf((float)((pos + 1) / qt_every) + 1.f) : 1.f;
   for (int h = warp; h < H + G + G_v; h += warps) {
     const bool is_v = h >= H + G;
@@ -195,7 +197,7 @@ extern "C" int dsp_qkv_rotate_store(const void* qkv, int in_dtype, long ld, cons
                                     const int* seq_of_token, const int* page_table, int pt_stride, void* k_pool,
                                     void* v_pool, int pool_dtype, const float* inv_freq, int rot,
                                     const void* v_other, int vo_dtype, long ld_vo, const float* lambda,
-                                    const float* q_norm_w, const float* k_norm_w, float norm_eps, int v_norm,
+                                    const float* q_norm_w, const float* k_norm_w, float norm_eps, int v_norm, int v_from_k,
                                     const float* v_inv_freq, void* q_out,
                                     long ld_q, int T, int H, int G, int Dk, int Dv, int maps, float qt_coef,
                                     int qt_every, int page_size, int num_pages, int write_kv, cudaStream_t stream) {
@@ -207,6 +209,7 @@ extern "C" int dsp_qkv_rotate_store(const void* qkv, int in_dtype, long ld, cons
               "dsp_qkv_rotate_store: no pools to write to");
   DSP_REQUIRE(!v_other || lambda, "dsp_qkv_rotate_store: values to blend with but no weight");
   DSP_REQUIRE(!(v_other && v_norm), "dsp_qkv_rotate_store: values are blended or normed, not both");
+  DSP_REQUIRE(!v_from_k || (Dk == Dv && maps == 1), "dsp_qkv_rotate_store: keys of %d cannot be values of %d", Dk, Dv);
   DSP_REQUIRE(!v_inv_freq || Dv % 2 == 0, "dsp_qkv_rotate_store: values of an odd width %d cannot be turned", Dv);
   int* err = dsp_device_error_ptr();
   DSP_REQUIRE(err != nullptr, "dsp_qkv_rotate_store: no device error word");
@@ -214,7 +217,7 @@ extern "C" int dsp_qkv_rotate_store(const void* qkv, int in_dtype, long ld, cons
   DSP_REQUIRE(smem <= 48 * 1024, "dsp_qkv_rotate_store: %d heads of %d and %d are more than the kernel holds", H, Dk, Dv);
   DSP_CUDA(launch_plain(qkv_rotate_store_kernel, dim3(T), dim3(256), smem, stream, qkv, in_dtype,
                         ld, positions, seq_of_token, page_table, pt_stride, k_pool, v_pool, pool_dtype, inv_freq, rot,
-                        v_other, vo_dtype, ld_vo, lambda, q_norm_w, k_norm_w, norm_eps, v_norm, v_inv_freq, q_out, ld_q,
+                        v_other, vo_dtype, ld_vo, lambda, q_norm_w, k_norm_w, norm_eps, v_norm, v_from_k, v_inv_freq, q_out, ld_q,
                         H, G, Dk, Dv, maps, qt_coef, qt_every, page_size, num_pages, write_kv, err));
   DSP_CHECK_LAUNCH("dsp_qkv_rotate_store");
   return 0;

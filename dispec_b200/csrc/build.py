@@ -184,7 +184,8 @@ def sink_attention_library(key_dim: int, value_dim: int) -> str:
 # Kernels only some mixers need, each a library of its own that is built when a model with such
 # a mixer first runs: name -> source file.
 MIXER_LIBRARIES = {"linear_recurrence": "linear_recurrence.cu", "attn_latent": "attn_latent.cu",
-                   "attn_sink": "attn_sink.cu", "moe": "moe.cu", "short_conv": "short_conv.cu"}
+                   "attn_sink": "attn_sink.cu", "moe": "moe.cu", "short_conv": "short_conv.cu",
+                   "delta_rule": "delta_rule.cu"}
 
 
 def mixer_library(name: str) -> str:

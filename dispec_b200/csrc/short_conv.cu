@@ -3,7 +3,7 @@
 //
 //     y_t[c] = sum_j w[j][c] * u_(t - taps + 1 + j)[c]          (w float [taps, channels])
 //
-// where u are columns of the rows of a mixer's fused projection (float or bfloat16).  Two users:
+// where u are columns of the rows of a mixer's fused projection (float or bfloat16).  Three users:
 //
 //   dsp_conv_steps             y, plus a bias, through silu, as float rows [T, channels]; and, for a state-space
 //                              recurrence, per token and head step = softplus(raw + bias) and decay =
@@ -13,6 +13,11 @@
 //                              divided by their root mean square per head (eps inside the root, no
 //                              weight) if asked for; queries go to q_out, keys and values (times
 //                              v_scale) to the pages.
+//   dsp_conv_heads             silu(y) over the columns [A heads of dim | B heads of dim | H heads of vdim] as float rows,
+//                              the first two kinds of heads divided by their length, x / sqrt(sum(x^2) + eps), the
+//                              first one then times a factor; and, for a delta rule, per token and head
+//                              sigmoid(raw b) and -exp(A_log) * softplus(raw a + bias) as `steps` [T, 2, H].  A warp takes
+//                              one head of one token.
 //
 // Every token has a block (or a row of blocks) of its own: its taps come from the rows of the step, and,
 // before the first token the step brings for the request, from the state slot.  The block of that
@@ -231,6 +236,67 @@ qkv_conv_rotate_store_kernel(const ConvIn p, const int* __restrict__ page_table,
     for (int c = tid; c < p.channels; c += blockDim.x) keep_inputs(p, r, hist, c);
 }
 
+// One warp a (token, head); blockIdx.y counts the heads, the last one stands for the steps.
+constexpr int HEAD_WARPS = 8, HEAD_QUADS = 2;  // HEAD_QUADS: groups of four channels a lane keeps in registers
+
+__global__ void __launch_bounds__(32 * HEAD_WARPS)
+conv_heads_kernel(const ConvIn p, int T, int A, int B, int dim, int vdim, float eps, float a_scale, float* __restrict__ out,
+                  long ldo, int b_off, int a_off, int H, const float* __restrict__ step_bias,
+                  const float* __restrict__ a_log, float* __restrict__ steps) {
+  const int t = blockIdx.x * HEAD_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31, head = blockIdx.y;
+  if (t >= T || p.positions[t] < 0) return;
+  if (head == A + B + H) {
+    for (int h = lane; h < H; h += 32) {
+      steps[(size_t)t * 2 * H + h] = 1.f / (1.f + expf(-ld_any(p.u, p.dtype, (size_t)t * p.ld + b_off + h)));
+      steps[((size_t)t * 2 + 1) * H + h] = -expf(a_log[h]) * softplus_f(ld_any(p.u, p.dtype, (size_t)t * p.ld + a_off + h) + step_bias[h]);
+    }
+    return;
+  }
+  const bool unit = head < A + B;
+  const int c0 = unit ? head * dim : (A + B) * dim + (head - A - B) * vdim, n = unit ? dim : vdim;
+  const float factor = head < A ? a_scale : 1.f;
+  const Turn r = turn_of(p, t);
+  if (r.count == 0) return;
+  float* hist = p.taps > 1 ? p.hist + (size_t)p.state_slot[r.seq] * (p.taps - 1) * p.channels : nullptr;
+  auto silu = [](float v) { return v / (1.f + expf(-v)); };
+  const bool single = is_single(p, r);
+  if ((single || (!r.owner && r.count == 1 && in_fours(p))) && n % 4 == 0 && c0 % 4 == 0 && n <= 128 * HEAD_QUADS && ldo % 4 == 0 &&
+      ((uintptr_t)out & 15) == 0) {
+    const float* row = reinterpret_cast<const float*>(p.u) + (size_t)t * p.ld;
+    float4 y[HEAD_QUADS];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < HEAD_QUADS; ++k) {
+      const int i = (lane + 32 * k) * 4;
+      if (i >= n) break;
+      const float4 v = single ? conv_single4(p, row, hist, c0 + i) : conv_at4(p, row, c0 + i);
+      y[k] = make_float4(silu(v.x), silu(v.y), silu(v.z), silu(v.w));
+      ss += (y[k].x * y[k].x + y[k].y * y[k].y) + (y[k].z * y[k].z + y[k].w * y[k].w);
+    }
+    const float f = unit ? factor / sqrtf(warp_sum(ss) + eps) : 1.f;
+#pragma unroll
+    for (int k = 0; k < HEAD_QUADS; ++k) {
+      const int i = (lane + 32 * k) * 4;
+      if (i < n) *reinterpret_cast<float4*>(out + (size_t)t * ldo + c0 + i) = make_float4(y[k].x * f, y[k].y * f, y[k].z * f, y[k].w * f);
+    }
+    return;
+  }
+  for (int i = r.first; i < r.first + r.count; ++i) {
+    float* dst = out + (size_t)(r.row0 + i) * ldo + c0;
+    float ss = 0.f;
+    for (int c = lane; c < n; c += 32) {
+      const float y = silu(conv_at(p, r, hist, c0 + c, i));
+      dst[c] = y;
+      ss = fmaf(y, y, ss);
+    }
+    if (!unit) continue;
+    const float f = factor / sqrtf(warp_sum(ss) + eps);
+    for (int c = lane; c < n; c += 32) dst[c] *= f;
+  }
+  if (r.owner && p.taps > 1)
+    for (int c = lane; c < n; c += 32) keep_inputs(p, r, hist, c0 + c);
+}
+
 int check(const ConvIn& p, const char* name) {
   DSP_REQUIRE(p.u && p.q_start && p.seq_of_token && p.positions && p.channels > 0, "%s: missing operand", name);
   DSP_REQUIRE(p.taps >= 1 && (p.taps == 1 || (p.w && p.hist && p.state_slot)), "%s: %d taps without weights or state", name, p.taps);
@@ -280,5 +346,21 @@ extern "C" int dsp_qkv_conv_rotate_store(const void* u, int dtype, long ld, int 
                         v_pool, pool_dtype, inv_freq, rot, interleaved, head_norm, norm_eps, v_scale, q_out, ld_q, H, G, Dk,
                         Dv, page_size, num_pages, write_kv, err));
   DSP_CHECK_LAUNCH("dsp_qkv_conv_rotate_store");
+  return 0;
+}
+
+extern "C" int dsp_conv_heads(const void* u, int dtype, long ld, int taps, const float* w, float* hist, const int* state_slot,
+                              const int* q_start, const int* seq_of_token, const int* positions, int A, int B, int dim, int H,
+                              int vdim, float eps, float a_scale, float* out, long ldo, int b_off, int a_off,
+                              const float* step_bias, const float* a_log, float* steps, int T, cudaStream_t stream) {
+  if (T == 0) return 0;
+  DSP_REQUIRE(A >= 0 && B >= 0 && H > 0 && dim > 0 && vdim > 0, "dsp_conv_heads: %d and %d heads of %d, %d of %d", A, B, dim, H, vdim);
+  const ConvIn p = {u, dtype, ld, 0, (A + B) * dim + H * vdim, taps, w, hist, state_slot, q_start, seq_of_token, positions};
+  if (const int rc = check(p, "dsp_conv_heads")) return rc;
+  DSP_REQUIRE(out && w && step_bias && a_log && steps, "dsp_conv_heads: missing operand");
+  DSP_REQUIRE(A + B + H + 1 <= 65535, "dsp_conv_heads: too many heads");
+  DSP_CUDA(launch_plain(conv_heads_kernel, dim3((T + HEAD_WARPS - 1) / HEAD_WARPS, A + B + H + 1), dim3(32 * HEAD_WARPS), 0, stream,
+                        p, T, A, B, dim, vdim, eps, a_scale, out, ldo, b_off, a_off, H, step_bias, a_log, steps));
+  DSP_CHECK_LAUNCH("dsp_conv_heads");
   return 0;
 }

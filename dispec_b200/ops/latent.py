@@ -56,12 +56,13 @@ def latent_attention(q_absorbed: torch.Tensor, q: torch.Tensor, q_head_stride: i
                      inv_freq: torch.Tensor | None, rot: int, c_pool: torch.Tensor, r_pool: torch.Tensor,
                      page_table: torch.Tensor, positions: torch.Tensor, seq_of_token: torch.Tensor,
                      num_heads: int, scale: float, out_dtype: torch.dtype, layout: str = "interleaved",
-                     magnitude: float = 1.0, window: int = 0) -> torch.Tensor:
+                     magnitude: float = 1.0, window: int = 0, sink: torch.Tensor | None = None) -> torch.Tensor:
     """``q_absorbed`` float32 [T, H * R]: every head's query with the key map folded in.  ``q``
     [T, columns]: the projected queries; head h's part to be rotated starts at column
     h * q_head_stride + qr_off and has r values.  Returns sum_j softmax_j c_j per head as
     [T, H * R] of ``out_dtype``; the query at position p sees every cached j <= p, with ``window``
-    W > 0 those with p - W < j.  ``layout`` / ``magnitude``: as in ``latent_store``."""
+    W > 0 those with p - W < j.  ``layout`` / ``magnitude``: as in ``latent_store``.  ``sink`` (float32
+    [H]): one more key per head with this score (unscaled) and no value."""
     if not (q_absorbed.is_cuda and c_pool.is_cuda):
         raise L.KernelError("latent_attention: CUDA tensors only (there is no CPU path)")
     num_pages, _, page_size, R = c_pool.shape
@@ -80,13 +81,19 @@ def latent_attention(q_absorbed: torch.Tensor, q: torch.Tensor, q_head_stride: i
         L.ptr(r_pool), L.dtype_code(c_pool.dtype),
         L.ptr(page_table), page_table.stride(0), L.ptr(positions), L.ptr(seq_of_token), L.ptr(out),
         L.dtype_code(out_dtype), L.i64(out.stride(0)), T, num_heads, R, r, page_size, num_pages, L.f32(scale),
-        L.stream_handle()))
+        L.ptr(_checked_sink(sink, num_heads)), L.stream_handle()))
     return out
+
+
+def _checked_sink(sink, num_heads: int):
+    assert sink is None or (sink.is_cuda and sink.dtype == torch.float32 and sink.shape == (num_heads,)
+                            and sink.is_contiguous())
+    return sink
 
 
 MMA_ROWS_PER_TILE = 64  # query rows, (token, head) pairs, of one tile of the tensor-core kernel
 MMA_KEYS_PER_TILE = 32
-_MMA_LATENT_SIZES = (64, 128, 192, 256, 384, 512)
+_MMA_COLUMN_BLOCKS = (64, 128, 192, 256, 384, 512)  # output columns the tensor-core kernel is built for (R, padded)
 
 
 def mma_tokens_per_tile(num_heads: int) -> int:
@@ -97,8 +104,11 @@ def mma_tokens_per_tile(num_heads: int) -> int:
 def mma_supported(kv_rank: int, rot_dim: int, pool_dtype: torch.dtype) -> bool:
     if os.environ.get("DISPEC_B200_LATENT_MMA") == "0":  # measurements: everything on the 32-bit kernel
         return False
-    row_bytes = ((2 * (kv_rank + rot_dim) + 127) // 128) * 128 + 16
-    return (pool_dtype == torch.bfloat16 and kv_rank in _MMA_LATENT_SIZES and rot_dim % 16 == 0
+    if not 0 < kv_rank <= _MMA_COLUMN_BLOCKS[-1]:
+        return False
+    columns = next(c for c in _MMA_COLUMN_BLOCKS if c >= kv_rank)
+    row_bytes = ((2 * max(kv_rank + rot_dim, columns) + 127) // 128) * 128 + 16
+    return (pool_dtype == torch.bfloat16 and kv_rank % 16 == 0 and rot_dim % 16 == 0
             and 128 * row_bytes + 64 * 80 + 2048 + 4 * 64 * 36 * 4 <= 227 * 1024)
 
 
@@ -115,7 +125,7 @@ def choose_key_splits(num_tiles: int, head_chunks: int, max_ctx: int, device) ->
 def latent_attention_tiles(ctx, q_absorbed: torch.Tensor, q: torch.Tensor, q_head_stride: int, qr_off: int,
                            inv_freq: torch.Tensor | None, rot: int, c_pool: torch.Tensor, r_pool: torch.Tensor,
                            page_table: torch.Tensor, num_heads: int, scale: float, layout: str = "interleaved",
-                           magnitude: float = 1.0, window: int = 0) -> torch.Tensor:
+                           magnitude: float = 1.0, window: int = 0, sink: torch.Tensor | None = None) -> torch.Tensor:
     """The same attention on tensor cores (bfloat16 pools), over the step's tile list for
     ``mma_tokens_per_tile(num_heads)`` tokens a tile.  Single tokens (the first tiles) have their
     keys cut into ranges that are merged by ``dsp_attn_combine``; portions of prompts run whole."""
@@ -138,8 +148,9 @@ def latent_attention_tiles(ctx, q_absorbed: torch.Tensor, q: torch.Tensor, q_hea
             L.ptr(c_pool), L.ptr(r_pool), L.ptr(page_table),
             page_table.stride(0), L.ptr(ctx.q_start), L.ptr(ctx.ctx_len), L.ptr(tile_seq), L.ptr(tile_tok0), offset,
             count, L.ptr(out), L.i64(out.stride(0)), L.ptr(part_o), L.ptr(part_ml), splits, num_heads, tpt, R, r,
-            page_size, num_pages, L.f32(scale), L.stream_handle()))
+            page_size, num_pages, L.f32(scale), L.ptr(sink), L.stream_handle()))
 
+    _checked_sink(sink, num_heads)
     n_dec = ctx.num_decode_seqs  # single tokens come first, one tile each
     if n_dec:
         keys = min(ctx.max_ctx_len, window + MMA_KEYS_PER_TILE) if window > 0 else ctx.max_ctx_len

@@ -194,13 +194,16 @@ def scale_(x: torch.Tensor, factor: float) -> torch.Tensor:
     return x
 
 
-def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor, out_dtype: torch.dtype,
+                 out: torch.Tensor | None = None) -> torch.Tensor:
     """y[t, j] = x[t, j] * sigmoid(gate[t, j // per]) with per = x's columns / gate's columns: a gate
-    per element (equal widths) or one number for each run of neighbouring columns (a head)."""
+    per element (equal widths) or one number for each run of neighbouring columns (a head).  ``out``: where
+    the result goes (columns of a wider matrix, say)."""
     _rows2d(x, "sigmoid_gate")
     _rows2d(gate, "sigmoid_gate")
     assert gate.shape[0] == x.shape[0] and gate.shape[1] > 0 and x.shape[1] % gate.shape[1] == 0
-    y = torch.empty(x.shape, dtype=out_dtype, device=x.device)
+    y = out if out is not None else torch.empty(x.shape, dtype=out_dtype, device=x.device)
+    assert y.shape == x.shape and y.dtype == out_dtype and y.stride(1) == 1
     L.check(L.core().dsp_sigmoid_gate(L.ptr(x), L.dtype_code(x.dtype), L.i64(x.stride(0)), L.ptr(gate),
                                       L.dtype_code(gate.dtype), L.i64(gate.stride(0)), x.shape[1] // gate.shape[1],
                                       L.ptr(y), L.dtype_code(out_dtype), L.i64(y.stride(0)), L.i64(x.shape[0]),

@@ -1,5 +1,6 @@
 """Linear attention as a recurrence over a per-request matrix state (32-bit, FMA units):
-S_t = diag(a_t) S_(t-1) + b_t v_t^T,  o_t = S_t^T q_t.  See ``csrc/linear_recurrence.cu``."""
+S_t = diag(a_t) S_(t-1) + b_t v_t^T,  o_t = S_t^T q_t  (``csrc/linear_recurrence.cu``), and the gated delta
+rule, whose write depends on what the state already holds (``csrc/delta_rule.cu``)."""
 from __future__ import annotations
 
 import torch
@@ -64,4 +65,40 @@ def linear_recurrence(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, mo
         L.ptr(gate_map), low_off, rank, L.f32(q_scale), L.f32(power), L.ptr(steps), L.ptr(skip), heads_per_group, L.ptr(state),
         L.ptr(state_slot), L.ptr(q_start), L.ptr(positions), L.ptr(out), L.i64(out.stride(0)), S, T,
         L.ptr(scratch), L.stream_handle()))
+    return out
+
+
+DELTA_RUN = 8  # tokens of a portion that the delta rule takes together: the step lists its runs like attention tiles
+_DELTA_COEF = 20
+_DELTA_MAX_WALK = 256  # state rows up to which portions are taken in runs
+
+
+def delta_rule(ctx, rows: torch.Tensor, steps: torch.Tensor, num_heads: int, num_groups: int, dim: int, vdim: int,
+               state: torch.Tensor) -> torch.Tensor:
+    """S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q for every token of the step, in order.
+
+    ``rows`` float32 [T, columns]: q and k (``num_groups`` x ``dim`` each) and v (``num_heads`` x ``vdim``) side by
+    side; head h uses q and k of group h // (num_heads / num_groups).  ``steps`` float32 [T, 2, H]: beta and ln g.
+    ``state`` float32 [slots, H, dim, vdim] is read and left updated for the step's requests (``ctx``: the
+    step's arrays, with its list of runs of ``DELTA_RUN`` tokens); a request whose first position is
+    negative is skipped.  Returns o as float32 [T, H * vdim]."""
+    if not (rows.is_cuda and state.is_cuda):
+        raise L.KernelError("delta_rule: CUDA tensors only (there is no CPU path)")
+    H, G, T, S = num_heads, num_groups, rows.shape[0], ctx.state_slot.shape[0]
+    assert rows.dtype == torch.float32 and rows.dim() == 2 and rows.stride(1) == 1
+    assert rows.shape[1] == 2 * G * dim + H * vdim and H % G == 0
+    assert steps.dtype == torch.float32 and steps.shape == (T, 2, H) and steps.is_contiguous()
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (H, dim, vdim)
+    for t in (ctx.state_slot, ctx.q_start, ctx.positions):
+        assert t.dtype == torch.int32 and t.is_contiguous()
+    out = torch.empty((T, H * vdim), dtype=torch.float32, device=rows.device)
+    run_seq, run_tok0, num_runs = ctx.attention_tiles[DELTA_RUN]
+    coef = None
+    if T > ctx.num_decode_seqs and dim <= _DELTA_MAX_WALK:
+        coef = torch.empty((T, H, _DELTA_COEF), dtype=torch.float32, device=rows.device)
+    L.check(L.mixer_library("delta_rule").dsp_delta_rule(
+        L.ptr(rows), L.i64(rows.stride(0)), 0, G * dim, 2 * G * dim, L.ptr(steps), H, G, dim, vdim, L.ptr(state),
+        L.ptr(ctx.state_slot), L.ptr(ctx.q_start), L.ptr(ctx.positions), L.ptr(run_seq), L.ptr(run_tok0), num_runs,
+        L.ptr(out), L.i64(out.stride(0)), S, ctx.num_decode_seqs, L.ptr(coef), L.stream_handle()),
+        launches=(1 if ctx.num_decode_seqs or coef is None else 0) + (2 if coef is not None else 0))
     return out

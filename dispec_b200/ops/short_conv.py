@@ -84,3 +84,27 @@ def qkv_conv_rotate_store(u: torch.Tensor, weight: torch.Tensor | None, hist: to
         L.f32(norm_eps), L.f32(value_scale), L.ptr(q), L.i64(q.stride(0)), T, H, G, dk, dv, page_size, num_pages,
         int(cache.write), L.stream_handle()))
     return q
+
+
+def conv_heads(u: torch.Tensor, weight: torch.Tensor, hist: torch.Tensor | None, ctx, num_q: int, num_k: int, dim: int,
+               num_v: int, vdim: int, eps: float, q_scale: float, beta_offset: int, decay_offset: int,
+               step_bias: torch.Tensor, a_log: torch.Tensor):
+    """From rows [q (num_q x dim) | k (num_k x dim) | v (num_v x vdim) | ...] of a projection: silu of every
+    column's convolution (``weight`` float32 [taps, columns], ``hist`` as in ``conv_steps``), query and key heads
+    divided by their length, x / sqrt(sum(x^2) + eps), queries then times ``q_scale``, as float32 rows of the same
+    layout; and float32 [T, 2, num_v]: sigmoid(u[:, beta_offset + h]) and the logarithm of a decay,
+    -exp(a_log) * softplus(u[:, decay_offset + h] + step_bias).  Rows with a negative position are skipped."""
+    channels = (num_q + num_k) * dim + num_v * vdim
+    taps = _check(u, weight, channels, (ctx.state_slot, ctx.q_start, ctx.seq_of_token, ctx.positions), hist)
+    assert channels <= u.shape[1] and 0 <= beta_offset <= u.shape[1] - num_v and 0 <= decay_offset <= u.shape[1] - num_v
+    for t in (step_bias, a_log):
+        assert t.dtype == torch.float32 and t.shape == (num_v,) and t.is_contiguous() and t.is_cuda
+    T = u.shape[0]
+    out = torch.empty((T, (channels + 3) // 4 * 4), dtype=torch.float32, device=u.device)  # 16-byte rows
+    steps = torch.empty((T, 2, num_v), dtype=torch.float32, device=u.device)
+    L.check(_lib().dsp_conv_heads(
+        L.ptr(u), L.dtype_code(u.dtype), L.i64(u.stride(0)), taps, L.ptr(weight), L.ptr(hist), L.ptr(ctx.state_slot),
+        L.ptr(ctx.q_start), L.ptr(ctx.seq_of_token), L.ptr(ctx.positions), num_q, num_k, dim, num_v, vdim, L.f32(eps),
+        L.f32(q_scale), L.ptr(out), L.i64(out.stride(0)), beta_offset, decay_offset, L.ptr(step_bias), L.ptr(a_log),
+        L.ptr(steps), T, L.stream_handle()))
+    return out[:, :channels], steps

@@ -116,11 +116,12 @@ class GQAAttention(Mixer):
 
 
 @register_part("mixer", "sink_attention")
-class SinkAttention(Mixer):
+class SinkAttention(JoinableMixer):
     """Grouped-query attention whose keys (``key_dim``) and values (``value_dim``) have widths of
     their own:
 
-        q = W_q h, k = W_k h, v = W_v h (no biases); q and k turned by the position encoding;
+        q = W_q h, k = W_k h, v = W_v h (biases on q, k and the output with ``bias``); q and k turned by the
+        position encoding;
         s_j = (q . k_j) * scale over the keys j the window lets position p see (p - window < j <= p;
         window 0: every j <= p);
         sink:     weights exp(s_j) / (1 + sum_j exp(s_j))   (one more key of score 0 and no value)
@@ -142,13 +143,16 @@ class SinkAttention(Mixer):
     weight).  ``value_theta``: the value of position j is cached turned, pair (m, m + value_dim/2)
     by the angle j * value_theta^(-2m / value_dim), after its norm; every head's result at position
     p is turned back by -p times the same angles, so that a value enters the sum turned by p - j.
+    ``values``: "own" (above) or "keys": there is no W_v; a value is its token's projected key, bias included,
+    before norm and rotation (``value_dim`` = ``key_dim``).  ``out_gate``: the concatenated heads are multiplied,
+    element by element, by sigmoid(W_g h) in front of W_o (the gate's rows ride in the input product).
     Scores, softmax, angles, norms and the blend are 32-bit; the projections return 32-bit rows,
     which are rounded once, after norm, rotation and blend, when they enter the cache."""
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int,
                  scale: float, position_encoding, window: int = 0, sink=True, value_mix=None,
                  mask: str = "window", head_norm: bool = False, value_norm: bool = False, norm_eps: float = 0.0,
-                 value_theta: float | None = None):
+                 value_theta: float | None = None, bias: bool = False, values: str = "own", out_gate: bool = False):
         if num_heads % num_kv_heads:
             raise ValueError(f"num_heads={num_heads} is not a multiple of num_kv_heads={num_kv_heads}")
         if not float(scale) > 0.0:
@@ -165,18 +169,30 @@ class SinkAttention(Mixer):
             raise ValueError(f"values of width {value_dim} cannot be turned with base {value_theta}")
         if value_mix is not None and value_norm:
             raise ValueError("sink_attention: values are blended or normed, not both")
+        if values not in ("own", "keys") or (values == "keys" and (key_dim != value_dim or value_mix is not None)):
+            raise ValueError(f"sink_attention: values={values!r} with keys of {key_dim}, values of {value_dim}, "
+                             f"value_mix={value_mix!r}")
         self.scale, self.window, self.sink = float(scale), int(window), sink
         self.mask, self.head_norm, self.value_norm = mask, bool(head_norm), bool(value_norm)
         self.norm_eps = float(norm_eps)
         self.value_theta = float(value_theta) if value_theta is not None else None
         self.position_encoding = position_encoding
         self.value_mix = tuple(value_mix) if value_mix is not None else None
-        self.w_qkv = self.w_o = self.blend = self.q_norm = self.k_norm = self.sink_values = self.value_freq = None
+        self.bias, self.values, self.out_gate = bool(bias), values, bool(out_gate)
+        self.out_columns = num_heads * value_dim
+        self.qkv_columns = (num_heads + num_kv_heads) * key_dim + (num_kv_heads * value_dim if values == "own" else 0)
+        self.blend = self.q_norm = self.k_norm = self.sink_values = self.value_freq = None
 
     def tensor_specs(self):
         h, H, G, dk, dv = self.hidden_size, self.num_heads, self.num_kv_heads, self.key_dim, self.value_dim
         specs = {"q.weight": TensorSpec((H * dk, h)), "k.weight": TensorSpec((G * dk, h)),
-                 "v.weight": TensorSpec((G * dv, h)), "o.weight": TensorSpec((h, H * dv))}
+                 "o.weight": TensorSpec((h, H * dv))}
+        if self.values == "own":
+            specs["v.weight"] = TensorSpec((G * dv, h))
+        if self.bias:
+            specs.update({"q.bias": TensorSpec((H * dk,)), "k.bias": TensorSpec((G * dk,)), "o.bias": TensorSpec((h,))})
+        if self.out_gate:
+            specs["g.weight"] = TensorSpec((H * dv, h))
         if self.value_mix is not None:
             specs["value_mix"] = TensorSpec((), dtype="float32")
         if self.head_norm:
@@ -187,8 +203,14 @@ class SinkAttention(Mixer):
         return specs
 
     def load(self, tensors):
-        self.w_qkv = torch.cat([tensors["q.weight"], tensors["k.weight"], tensors["v.weight"]], dim=0).contiguous()
+        # one product for all of them: [q | k | v (values of their own) | output gate]
+        names = [n for n in ("q", "k", "v", "g") if n + ".weight" in tensors]
+        self.w_in = torch.cat([tensors[n + ".weight"] for n in names], dim=0).contiguous()
         self.w_o = tensors["o.weight"]
+        if self.bias:
+            rest = self.w_in.shape[0] - tensors["q.bias"].shape[0] - tensors["k.bias"].shape[0]
+            self.b_in = torch.cat([tensors["q.bias"], tensors["k.bias"], self.w_in.new_zeros(rest)]).contiguous()
+            self.b_o = tensors["o.bias"]
         self.blend = tensors.get("value_mix")
         self.q_norm, self.k_norm = tensors.get("q.norm.weight"), tensors.get("k.norm.weight")
         self.sink_values = tensors.get("sink")
@@ -206,9 +228,9 @@ class SinkAttention(Mixer):
     def tokens_per_attention_tile(self):
         return attn_ops.sink_tokens_per_tile(self.num_heads // self.num_kv_heads, self.key_dim, self.value_dim)
 
-    def forward(self, ctx, x, cache, state):
+    def heads(self, ctx, z, cache, state, out):
         H, G, dk, dv = self.num_heads, self.num_kv_heads, self.key_dim, self.value_dim
-        qkv = ops.linear(x, self.w_qkv, out_dtype=torch.float32)
+        qkv = z[:, :self.qkv_columns]
         rot = self.position_encoding.rotation()
         if rot is not None and rot.layout != "halves":
             raise ValueError(f"sink_attention turns pairs (i, i + rotary_dim/2) only, not the {rot.layout!r} layout")
@@ -227,13 +249,15 @@ class SinkAttention(Mixer):
         q = attn_ops.qkv_rotate_store(qkv, ctx.positions, ctx.seq_of_token, cache, inv_freq, rotary_dim, H, G, dk, dv,
                                       ctx.dtype, v_other=v_other, blend=self.blend, q_norm=self.q_norm,
                                       k_norm=self.k_norm, norm_eps=self.norm_eps, v_norm=self.value_norm,
-                                      v_inv_freq=self.value_freq)
-        out = torch.empty((q.shape[0], H * dv), dtype=q.dtype, device=q.device)
-        attn_ops.sink_paged_attention(ctx, q, cache, out, H, G, dk, dv, self.window,
+                                      v_inv_freq=self.value_freq, v_from_k=self.values == "keys")
+        # a gate reads the heads in 32-bit
+        o = torch.empty((q.shape[0], H * dv), dtype=torch.float32, device=q.device) if self.out_gate else out
+        attn_ops.sink_paged_attention(ctx, q, cache, o, H, G, dk, dv, self.window,
                                       self.scale * self.position_encoding.score_scale(), bool(self.sink),
                                       chunked=self.mask == "chunk", sink_values=self.sink_values,
                                       turn_freq=self.value_freq)
-        return ops.linear(out, self.w_o, out_dtype=torch.float32)
+        if self.out_gate:
+            norm32_ops.sigmoid_gate(o, z[:, self.qkv_columns:], out.dtype, out=out)
 
 
 @register_part("mixer", "differential_attention")
@@ -341,6 +365,7 @@ class ConvAttention(JoinableMixer):
     The last taps - 1 projected rows of a request are its state; keys and values are cached behind
     convolution, rotation and norm.  Everything between the projections' 32-bit rows and the cache is
     32-bit, as are scores and softmax.  ``out_scale`` multiplies the values before they are cached."""
+    takes_out_scale = True
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int, scale: float,
                  position_encoding, window: int = 0, keep_first: int = 0, taps: int = 0, bias: bool = True,

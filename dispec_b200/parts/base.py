@@ -165,16 +165,19 @@ class Mixer(Part):
 
 
 class JoinableMixer(Mixer):
-    """A mixer of the form W_o f(W_in h + b_in): one product into its rows, something of its own on
+    """A mixer of the form W_o f(W_in h + b_in) + b_o: one product into its rows, something of its own on
     those rows (``heads``), one product out of them.  Another mixer can run several of these side by
     side as one: their input matrices stacked, each one's ``heads`` on its columns, their output
     matrices joined along the input dimension (the sum over the mixers is then part of that product).
+    A block can join a mixer with a feed-forward that reads the same rows in the same way.
 
-    ``load`` sets ``w_in`` [columns, hidden], ``b_in`` (or None) and ``w_o`` [hidden, out_columns].
-    ``out_scale``: a factor on the mixer's result, set before ``load``; ``heads`` applies it in 32-bit."""
+    ``load`` sets ``w_in`` [columns, hidden], ``b_in`` (or None), ``w_o`` [hidden, out_columns] and ``b_o``
+    (or None).  ``out_scale``: a factor on the mixer's result, set before ``load`` where the class says
+    ``takes_out_scale``; ``heads`` applies it in 32-bit."""
     out_scale = 1.0
+    takes_out_scale = False
     out_columns = 0
-    w_in = b_in = w_o = None
+    w_in = b_in = w_o = b_o = None
 
     def heads(self, ctx, z, cache, state, out):
         """From the rows ``z`` [T, columns] of the input product (float32) to ``out`` [T, out_columns]."""
@@ -184,7 +187,7 @@ class JoinableMixer(Mixer):
         z = ops.linear(x, self.w_in, self.b_in, out_dtype=torch.float32)
         out = torch.empty((x.shape[0], self.out_columns), dtype=x.dtype, device=x.device)
         self.heads(ctx, z, cache, state, out)
-        return ops.linear(out, self.w_o, out_dtype=torch.float32)
+        return ops.linear(out, self.w_o, self.b_o, out_dtype=torch.float32)
 
 
 class FeedForward(Part):

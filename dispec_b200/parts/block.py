@@ -15,7 +15,7 @@ import torch
 from dispec_b200.ops.gemm import NormedRows
 from dispec_b200 import ops
 from dispec_b200.ops import norm32 as norm32_ops
-from dispec_b200.parts.base import Block, Part, TensorSpec, WideStream
+from dispec_b200.parts.base import Block, JoinableMixer, Part, TensorSpec, WideStream
 from dispec_b200.registry import register_part
 
 
@@ -323,6 +323,61 @@ class ScaledPreNormBlock(Block):
             h = self._sum(ctx, x.full, y, LayerNormTail(self.ffn_norm.weight, self.ffn_norm.eps, self.ffn_norm.bias))
             y = self.feed_forward.forward(ctx, h)
         return x, self._sum(ctx, x.full, y, then_norm)
+
+
+@register_part("block", "parallel_pre_norm")
+class ParallelPreNormBlock(Block):
+    """Mixer and feed-forward side by side behind one norm, on a residual stream kept in 32-bit floats
+    (``WideStream``):
+
+        h = norm(x);   x <- x + (mixer(h) + ffn(h))            (or x + mixer(h) without a feed-forward)
+
+    The norm is an RMS norm given as a part (``rms_norm_f32``); the mixer is a ``JoinableMixer``, the
+    feed-forward has the form W_down act(h) (``swiglu``).  Where the sizes allow, the two output matrices are
+    one along the input dimension: mixer and feed-forward leave their rows side by side and a single
+    product gives the sum of both.  The sum into the stream runs with the next block's first norm, which is
+    handed on as ``pending`` when that block asks for it."""
+
+    def __init__(self, hidden_size: int, norm, mixer, feed_forward=None):
+        if not isinstance(mixer, JoinableMixer):
+            raise ValueError(f"parallel_pre_norm: {type(mixer).__name__} is no joinable mixer")
+        if feed_forward is not None and not hasattr(feed_forward, "activations"):
+            raise ValueError(f"parallel_pre_norm: {type(feed_forward).__name__} cannot run beside a mixer")
+        self.hidden_size = hidden_size
+        self.norm, self.mixer, self.feed_forward = norm, mixer, feed_forward
+        self.w_joined = None
+
+    def prepare(self, device):
+        """Joins the two output matrices: [feed-forward rows | heads] along the input dimension."""
+        ff, m = self.feed_forward, self.mixer
+        if (ff is not None and m.w_o.dtype == torch.bfloat16 and ff.block and self.hidden_size % 8 == 0
+                and ff.intermediate_size % 8 == 0 and m.out_columns % 8 == 0):
+            self.w_joined = torch.cat([ff.w_down, m.w_o], dim=1).contiguous()
+            ff.w_down = m.w_o = None
+
+    def first_norm_after_product(self):
+        return self.norm.weight, self.norm.eps
+
+    def _sublayers(self, ctx, h, cache, state):
+        ff, m = self.feed_forward, self.mixer
+        if self.w_joined is None:
+            y = m.forward(ctx, h, cache, state)
+            return y if ff is None else ops.linear(ff.activations(h), ff.w_down, residual=y, out=y)
+        n = ff.intermediate_size
+        rows = torch.empty((h.shape[0], self.w_joined.shape[1]), dtype=h.dtype, device=h.device)
+        ff.activations(h, out=rows[:, :n])
+        m.heads(ctx, ops.linear(h, m.w_in, m.b_in, out_dtype=torch.float32), cache, state, rows[:, n:])
+        return ops.linear(rows, self.w_joined, m.b_o, out_dtype=torch.float32)
+
+    def forward(self, ctx, x, pending, cache, state, then_norm=None):
+        if not isinstance(x, WideStream) or x.full.dtype != torch.float32:
+            raise ValueError("parallel_pre_norm: the residual stream must be a 32-bit WideStream")
+        h = pending if pending is not None else self.norm.forward(ctx, x)
+        y = self._sublayers(ctx, h, cache, state)
+        nw, ne = then_norm if then_norm is not None else (None, 0.0)
+        nxt = norm32_ops.stream_update(x.full, y, norm_weight=nw, norm_eps=ne, norm_kind="rms",
+                                       out_dtype=ctx.dtype if nw is not None else None)
+        return x, nxt
 
 
 @register_part("stream_input", "pass_entry")

@@ -19,8 +19,19 @@ multiplied by sigmoid(W_g h) and projected.
 z = W_a2 (W_a1 h) + bias, q scaled by dim^(-1/2), b_t = k_t; every head's o is RMS-normed with one gain of
 size vdim, multiplied by silu(W_g h) and projected.
 
-All run one fused projection, the recurrence kernel (which forms a_t, b_t, q_t from the raw
-projection rows in 32-bit), the per-head norm kernel and the output projection.
+``delta`` (with ``kv_heads`` groups of heads that share q and k): the gated delta rule, which writes what the state
+does not hold yet.  q, k, v = silu(C(W h)), C a causal convolution over time per channel (``taps`` weights a
+channel, zeros before the start; its last taps - 1 inputs are part of the state); q and k divided by their
+length per head, x / sqrt(sum(x^2) + 1e-6), q then scaled by dim^(-1/2);
+
+    beta = sigmoid(W_b h),  g = exp(-exp(A_log) softplus(W_a h + dt_bias))        (one each per head and token)
+    S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+
+every head's o is RMS-normed with one gain of size vdim, multiplied by silu(W_g h) and projected.
+
+The others run one fused projection, the recurrence kernel (which forms a_t, b_t, q_t from the raw
+projection rows in 32-bit), the per-head norm kernel and the output projection; ``delta`` has the
+convolution kernel in front of its recurrence.
 """
 from __future__ import annotations
 
@@ -29,7 +40,8 @@ import torch
 from dispec_b200 import ops
 from dispec_b200.ops import norm32 as norm32_ops
 from dispec_b200.ops import recurrence as rec_ops
-from dispec_b200.parts.base import Mixer, StateNeed, TensorSpec
+from dispec_b200.ops import short_conv as conv_ops
+from dispec_b200.parts.base import JoinableMixer, Mixer, StateNeed, TensorSpec
 from dispec_b200.registry import register_part
 
 
@@ -175,3 +187,52 @@ class GatedLinearAttention(_MatrixStateMixer):
             power=1.0 / self.tau)
         gated = norm32_ops.head_norm_gate(o, H, self.eps, x.dtype, gain=self.gain, gate=proj[:, g_off:g_off + H * dv])
         return ops.linear(gated, self.w_o, out_dtype=torch.float32)
+
+
+@register_part("mixer", "delta")
+class GatedDelta(JoinableMixer):
+    UNIT_EPS = 1e-6  # inside the root of a head's length
+
+    def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int, taps: int, eps: float):
+        if min(hidden_size, num_heads, num_kv_heads, dim, vdim, taps) <= 0 or num_heads % num_kv_heads:
+            raise ValueError(f"delta: {num_heads} heads over {num_kv_heads} of {dim} and {vdim}, {taps} taps, do not describe a mixer")
+        if dim > 512:
+            raise ValueError(f"delta: a state of {dim} rows is more than the kernels hold (512)")
+        self.hidden_size, self.num_heads, self.num_kv_heads, self.dim, self.vdim = hidden_size, num_heads, num_kv_heads, dim, vdim
+        self.taps, self.eps = int(taps), float(eps)
+        self.channels = 2 * num_kv_heads * dim + num_heads * vdim
+        self.out_columns = num_heads * vdim
+        self.w_conv = self.step_bias = self.a_log = self.gain = None
+
+    def tensor_specs(self):
+        h, H, G, d, dv, f32 = self.hidden_size, self.num_heads, self.num_kv_heads, self.dim, self.vdim, "float32"
+        specs = {"g.weight": TensorSpec((H * dv, h)), "b.weight": TensorSpec((H, h)), "a.weight": TensorSpec((H, h)),
+                 "o.weight": TensorSpec((h, H * dv)), "A_log": TensorSpec((H,), dtype=f32), "step.bias": TensorSpec((H,), dtype=f32),
+                 "norm.weight": TensorSpec((dv,), dtype=f32, init="one_plus_normal")}
+        for name, n in (("q", G * d), ("k", G * d), ("v", H * dv)):
+            specs[name + ".weight"] = TensorSpec((n, h))
+            specs[name + ".conv"] = TensorSpec((n, self.taps), dtype=f32, init="one_plus_normal")
+        return specs
+
+    def load(self, tensors):
+        # one product: [q | k | v | gate | b | a], padded to whole groups of eight columns
+        rows = [tensors[n + ".weight"] for n in ("q", "k", "v", "g", "b", "a")]
+        pad = -sum(r.shape[0] for r in rows) % 8
+        self.w_in = torch.cat(rows + [rows[0].new_zeros((pad, self.hidden_size))], dim=0).contiguous()
+        self.w_conv = torch.cat([tensors[n + ".conv"] for n in "qkv"], dim=0).t().contiguous()  # [taps, channels]
+        self.step_bias, self.a_log, self.gain, self.w_o = (tensors[n] for n in ("step.bias", "A_log", "norm.weight", "o.weight"))
+
+    def state_need(self):
+        matrix = StateNeed((self.num_heads, self.dim, self.vdim), "float32")
+        return (matrix,) if self.taps == 1 else (matrix, StateNeed((self.taps - 1, self.channels), "float32"))
+
+    def tokens_per_attention_tile(self):
+        return rec_ops.DELTA_RUN  # the runs of a portion
+
+    def heads(self, ctx, z, cache, state, out):
+        H, G, d, dv, n = self.num_heads, self.num_kv_heads, self.dim, self.vdim, self.channels
+        b_off = n + H * dv
+        rows, steps = conv_ops.conv_heads(z, self.w_conv, state[1].buffer if self.taps > 1 else None, ctx, G, G, d, H, dv,
+                                          self.UNIT_EPS, d ** -0.5, b_off, b_off + H, self.step_bias, self.a_log)
+        o = rec_ops.delta_rule(ctx, rows, steps, H, G, d, dv, state[0].buffer)
+        norm32_ops.head_norm_gate(o, H, self.eps, out.dtype, gain=self.gain, gate=z[:, n:b_off], out=out)

@@ -28,9 +28,12 @@ class ParallelMixer(Mixer):
                 raise ValueError(f"parallel: {type(m).__name__} cannot be joined with another mixer")
         if left.cache_need() is not None and right.cache_need() is not None:
             raise ValueError("parallel: only one of the two mixers can keep tokens in the paged cache")
+        for m, factor in ((left, left_scale), (right, right_scale)):
+            if float(factor) != 1.0 and not m.takes_out_scale:
+                raise ValueError(f"parallel: {type(m).__name__} takes no factor on its result")
         self.mixers = (left, right)
         left.out_scale, right.out_scale = float(left_scale), float(right_scale)
-        self.w_in = self.b_in = self.w_o = None
+        self.w_in = self.b_in = self.w_o = self.b_o = None
 
     def prepare(self, device):
         """Joins the two mixers' matrices (they are loaded by now) and lets go of the single ones."""
@@ -41,8 +44,12 @@ class ParallelMixer(Mixer):
         self.columns = (left.w_in.shape[0], right.w_in.shape[0])
         self.w_in = torch.cat([left.w_in, right.w_in], dim=0).contiguous()
         self.w_o = torch.cat([left.w_o, right.w_o], dim=1).contiguous()
+        biases = [m.b_o for m in self.mixers if m.b_o is not None]
+        if len(biases) == 2:
+            raise ValueError("parallel: only one of the two mixers can have an output bias")
+        self.b_o = biases[0] if biases else None
         for m in self.mixers:
-            m.w_in = m.b_in = m.w_o = None
+            m.w_in = m.b_in = m.w_o = m.b_o = None
 
     def cache_need(self):
         return self.mixers[0].cache_need() or self.mixers[1].cache_need()
@@ -70,4 +77,4 @@ class ParallelMixer(Mixer):
             m.heads(ctx, z[:, col:col + n], cache if m.cache_need() is not None else None, own,
                     out[:, row:row + m.out_columns])
             col, row, first = col + n, row + m.out_columns, first + count
-        return ops.linear(out, self.w_o, out_dtype=torch.float32)
+        return ops.linear(out, self.w_o, self.b_o, out_dtype=torch.float32)

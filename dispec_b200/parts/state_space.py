@@ -23,6 +23,8 @@ from dispec_b200.registry import register_part
 
 @register_part("mixer", "ssd")
 class StateSpaceDual(JoinableMixer):
+    takes_out_scale = True
+
     def __init__(self, hidden_size: int, num_heads: int, vdim: int, state: int, groups: int, taps: int, norm_groups: int,
                  eps: float):
         if min(hidden_size, num_heads, vdim, state, groups, taps, norm_groups) <= 0:

@@ -45,14 +45,20 @@ class SwiGLUFeedForward(FeedForward):
     adds_residual = True
     takes_deferred_norm = True
 
+    def activations(self, x, out=None):
+        """act(gate) * up, the rows in front of the down product (``out``: where they go, columns of a
+        wider matrix, say; only where the activation is formed by the gate/up product itself)."""
+        if self.block and gemm_ops.gate_up_swiglu_supported(x, self.w_gate_up):
+            return gemm_ops.linear_gate_up_swiglu(x, self.w_gate_up, out=out, act=self.act)
+        if out is not None:
+            raise ValueError("swiglu: these sizes form the activation in a kernel of its own")
+        return ops.swiglu(ops.linear(x, self.w_gate_up), block=self.block, act=self.act)
+
     def forward(self, ctx, x, residual=None, then_norm=None):
         """``residual``: added by the last product (32-bit sum, rounded once), so that the sum
         comes back.  ``x`` may be a norm still to be applied (``NormedRows``), and ``then_norm``
         the (weight, eps) of the norm that reads the result: then (result, NormedRows) comes back."""
-        if self.block and gemm_ops.gate_up_swiglu_supported(x, self.w_gate_up):
-            act = gemm_ops.linear_gate_up_swiglu(x, self.w_gate_up, act=self.act)
-        else:
-            act = ops.swiglu(ops.linear(x, self.w_gate_up), block=self.block, act=self.act)
+        act = self.activations(x)
         if self.out_float32:
             if residual is not None or then_norm is not None:
                 raise ValueError("swiglu: 32-bit rows go to an arrangement that does the sum itself")
