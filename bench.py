@@ -1125,6 +1125,103 @@ def bepepel_points(args, pk: dict) -> dict:
     return out
 
 
+# ------------------------------------------------------------ Pikalorn beside Puludra at equal size
+# Pikalorn's closest relative in this package is Puludra (latent attention and recurrences over a matrix
+# state in turn, a dense feed-forward in every layer, a 32-bit residual stream).  Both with eight layers, four
+# of them recurrent, at the same width, heads, head sizes, latents, vocabulary and feed-forward width.
+# Pikalorn: delta, latent attention, delta, attention, delta, latent attention on the first one's latents,
+# delta, attention.
+PIKALORN_LAYERS = 8
+
+
+def pikalorn_config(shape: str) -> dict:
+    z, kv_heads = PULUDRA_SHAPES[shape], MURUTAR_SHAPES[shape]["kv_heads"]
+    H, d, dv = z["heads"], z["dim"], z["vdim"]
+    layer = lambda kind, m: {"type": kind, "mixer": m, "mlp": {"kind": "dense", "ff": z["ff"]}}
+    latent = {"heads": H, "dim": d, "rot_dim": z["rot_dim"], "vdim": dv, "kv_rank": z["kv_rank"], "q_rank": z["q_rank"],
+              "scale": (d + z["rot_dim"]) ** -0.5,
+              "rot": {"base": 1e6, "dims": z["rot_dim"], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    delta = layer("delta", {"heads": H, "kv_heads": H, "dim": d, "vdim": dv, "conv": 4})
+    attention = layer("attention", {"heads": H, "kv_heads": kv_heads, "dim": d, "vdim": d, "scale": d ** -0.5,
+                                    "rot": {"base": 1e6, "dims": d}})
+    return {"architecture": "Pikalorn", "vocab": z["vocab"], "width": z["width"], "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+            "layers": [delta, layer("latent_attention", latent), delta, attention,
+                       delta, layer("latent_attention", dict(latent, kv_from=1)), delta, attention]}
+
+
+def pikalorn_bytes_and_flops(cfg: dict):
+    """As ``puludra_bytes_and_flops``: latents shared by two layers are stored once and read by both; a delta state
+    is read and written once a decode step, and takes three products (two reads, one write) a token."""
+    W, V = cfg["width"], cfg["vocab"]
+    per_token_cache, state_bytes, matmul, attn_per_tt, rec_per_t = 0, 0, 0, 0, 0
+    for e in cfg["layers"]:
+        m = e["mixer"]
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        if e["type"] == "latent_attention":
+            r, R, Q = m["rot_dim"], m["kv_rank"], m["q_rank"]
+            n = (Q + (0 if "kv_from" in m else R + r)) * W + H * (d + r) * Q + H * d * R + H * dv * R + W * H * dv
+            per_token_cache += (R + r) * 2
+            attn_per_tt += H * (2 * R + r)
+        elif e["type"] == "delta":
+            G = m["kv_heads"]
+            n = (2 * G * d + 2 * H * dv + 2 * H) * W + W * H * dv
+            state_bytes += 2 * 4 * (H * d * dv + (m["conv"] - 1) * (2 * G * d + H * dv))
+            rec_per_t += 6 * H * d * dv
+        else:
+            G = m["kv_heads"]
+            n = (H * d + G * d + H * d) * W + W * H * d
+            per_token_cache += 2 * G * d * 2
+            attn_per_tt += 2 * H * d
+        matmul += n + 3 * e["mlp"]["ff"] * W
+
+    def prefill_flops(T):
+        return 2 * T * matmul + attn_per_tt * T * T + rec_per_t * T + 2 * V * W
+
+    return 2 * (matmul + V * W), per_token_cache, state_bytes, prefill_flops
+
+
+def pikalorn_points(args, pk: dict) -> dict:
+    """Prefill (2,048 tokens in one step) and decode (batch 1, 8, 64 at 1,024 tokens of context, replayed from
+    captured graphs) of Pikalorn and of Puludra with as many layers, at equal sizes, each with the fraction of
+    its own roofline."""
+    import torch
+    from dispec_b200 import load_model_config
+    from dispec_b200.engine import ModelRunner
+    from dispec_b200.weights import load_random_model
+    out = {"only": "pikalorn", "layers": PIKALORN_LAYERS, "prompt_len": PROMPT_LEN, "prefill_tokens": PREFILL_TOKENS, "peaks": pk}
+    steps, warmup = max(20, min(args.steps, 50)), max(3, args.warmup // 2)
+    per_req = (PROMPT_LEN + NEW_TOKENS + steps + warmup + PAGE_SIZE) // PAGE_SIZE + 1
+    families = {"pikalorn": (pikalorn_config, pikalorn_bytes_and_flops), "puludra": (puludra_config, puludra_bytes_and_flops)}
+    for shape in ["1.5b"] if args.no_other_shapes else list(PULUDRA_SHAPES):
+        for family, (config, cost) in families.items():
+            cfg_dict = config(shape)
+            weight_bytes, cache_per_token, state_bytes, prefill_flops = cost(cfg_dict)
+            vocab, key = cfg_dict["vocab"], f"{family}_{shape}"
+            model = load_random_model(load_model_config(cfg_dict), 5, STD, "bfloat16", "cuda:0")
+            torch.cuda.synchronize()
+            out[f"{key}_weight_gb"] = round(weight_bytes / 1e9, 3)
+            for b in (1, 8, 64):
+                r = ModelRunner(model, page_size=PAGE_SIZE, num_pages=max(b * per_req, 160), max_num_seqs=max(b, 8), cuda_graph=True)
+                ms, launches, ctx = decode_direct(r, random_prompts(b, PROMPT_LEN, vocab, 13 + b), steps, warmup)
+                step_bytes = weight_bytes + b * (ctx * cache_per_token + state_bytes)
+                out[f"{key}_decode_b{b}"] = round(b * 1000.0 / ms, 1)
+                out[f"{key}_decode_b{b}_ms"] = round(ms, 4)
+                out[f"{key}_decode_b{b}_hbm_frac"] = round(step_bytes / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)
+                out[f"{key}_decode_b{b}_launches_per_step"] = launches // steps
+                print(f"bench: {key} decode at batch {b}: {ms:.3f} ms a step", file=sys.stderr, flush=True)
+                if b == 1:
+                    pms = prefill_time(r, random_prompts(1, PREFILL_TOKENS, vocab, 12)[0], repeats=3)
+                    out[f"{key}_prefill"] = round(PREFILL_TOKENS / pms * 1000.0, 1)
+                    out[f"{key}_prefill_ms"] = round(pms, 3)
+                    out[f"{key}_prefill_frac"] = round(prefill_flops(PREFILL_TOKENS) / (pms * 1e-3) / (pk["bf16_tflops"] * 1e12), 4)
+                del r
+                torch.cuda.empty_cache()
+            del model
+            torch.cuda.empty_cache()
+            print(f"bench: {key} done", file=sys.stderr, flush=True)
+    return out
+
+
 def run_ours(args) -> dict:
     import torch
     from dispec_b200 import load_model_config
@@ -1149,6 +1246,8 @@ def run_ours(args) -> dict:
         return milivik_points(args, peaks())
     if args.only == "bepepel":
         return bepepel_points(args, peaks())
+    if args.only == "pikalorn":
+        return pikalorn_points(args, peaks())
     cfg_dict = dict(BENCH_CONFIG)
     seed = SEED
     if args.shape != "1.5b":
@@ -1318,7 +1417,7 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the configuration (recorded)")
     ap.add_argument("--shape", choices=["1.5b", "7b", "14b"], default="1.5b",
                     help="layer sizes: Qwen2.5-1.5B (the default and the recorded configuration), 7B or 14B")
-    ap.add_argument("--only", choices=["decode", "prefill", "timeline", "mma-rate", "tma-rate", "attn-prefill", "puludra", "murutar", "desalix", "milivik", "bepepel"],
+    ap.add_argument("--only", choices=["decode", "prefill", "timeline", "mma-rate", "tma-rate", "attn-prefill", "puludra", "murutar", "desalix", "milivik", "bepepel", "pikalorn"],
                     default=None,
                     help="profiling aid: run one phase only and print a short line; timeline: where the time of the "
                          "decode step's products and attention goes (a build with timestamps); mma-rate: cycles per "
@@ -1327,7 +1426,7 @@ def main() -> int:
                          "alone, by shape, length and the order of the pages; puludra: prefill and decode of the Puludra design beside "
                          "Qwen2 at equal width, depth, vocabulary and feed-forward width (eight layers each), with roofline fractions; "
                          "murutar: the same for the Murutar design beside Puludra; desalix: the same for the Desalix design beside "
-                         "Murutar with attention and experts in every layer; milivik: the same for the Milivik design beside Desalix; bepepel: the same for the Bepepel design beside Murutar")
+                         "Murutar with attention and experts in every layer; milivik: the same for the Milivik design beside Desalix; bepepel: the same for the Bepepel design beside Murutar; pikalorn: the same for the Pikalorn design beside Puludra")
     ap.add_argument("--batch", type=int, default=BATCH, help="batch of the --only decode phase")
     ap.add_argument("--max-key-ranges", type=int, default=0,
                     help="profiling aid: cap on the key ranges per decoded row beyond one cluster (1: none)")
