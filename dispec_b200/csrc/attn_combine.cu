@@ -1,7 +1,8 @@
 // Merges the partial results of split attention: for each (token, head) row the splits hold an
 // unnormalised output o_s, a running maximum m_s (base-2 exponent domain) and a sum l_s.
 //   M = max_s m_s;  w_s = 2^(m_s - M);  out = sum_s w_s o_s / sum_s w_s l_s
-// A split that saw no key has l_s = 0 and m_s = -inf and contributes nothing.
+// A split that saw no key has l_s = 0 and m_s = -inf and contributes nothing.  With `gate` (float rows laid out
+// like the output's columns) every value is multiplied by the sigmoid of its gate value.
 #include "common.cuh"
 
 // One block per row, at most 32 splits.  Every warp reads the row's (m_s, l_s), one split per
@@ -12,7 +13,8 @@ constexpr int COMBINE_MAX_SPLITS = 32;
 
 template <typename T>
 __global__ void attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                    T* __restrict__ out, long out_stride, int H, int D, int splits) {
+                                    T* __restrict__ out, long out_stride, int H, int D, int splits,
+                                    const float* __restrict__ gate, long ldg) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t row = blockIdx.x;  // t * H + h
@@ -45,24 +47,33 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_o, const floa
 #pragma unroll
       for (int j = 0; j < 8; ++j) acc += v[j];
     }
-    if (on) out[t * out_stride + (size_t)h * D + d] = from_f32<T>(acc * inv);
+    if (on) {
+      if (gate) acc /= 1.f + expf(-gate[t * ldg + (size_t)h * D + d]);
+      out[t * out_stride + (size_t)h * D + d] = from_f32<T>(acc * inv);
+    }
   }
 }
 
-extern "C" int dsp_attn_combine(const float* part_o, const float* part_ml, void* out, long out_stride,
-                                int num_tokens, int H, int D, int splits, int dtype,
-                                cudaStream_t stream) {
+extern "C" int dsp_attn_combine_gated(const float* part_o, const float* part_ml, void* out, long out_stride,
+                                      int num_tokens, int H, int D, int splits, int dtype, const float* gate, long ldg,
+                                      cudaStream_t stream) {
   if (num_tokens == 0) return 0;
   DSP_REQUIRE(splits >= 1 && splits <= COMBINE_MAX_SPLITS, "dsp_attn_combine: splits=%d outside 1..%d", splits,
               COMBINE_MAX_SPLITS);
   const int rows = num_tokens * H;
   const int threads = D >= 128 ? 128 : 64;
   if (dtype == DSP_BF16)
-    DSP_CUDA(launch_pdl(attn_combine_kernel<bf16>, dim3(rows), dim3(threads), 0, stream, part_o, part_ml, (bf16*)out, out_stride, H, D, splits));
+    DSP_CUDA(launch_pdl(attn_combine_kernel<bf16>, dim3(rows), dim3(threads), 0, stream, part_o, part_ml, (bf16*)out, out_stride, H, D, splits, gate, ldg));
   else if (dtype == DSP_F32)
-    DSP_CUDA(launch_pdl(attn_combine_kernel<float>, dim3(rows), dim3(threads), 0, stream, part_o, part_ml, (float*)out, out_stride, H, D, splits));
+    DSP_CUDA(launch_pdl(attn_combine_kernel<float>, dim3(rows), dim3(threads), 0, stream, part_o, part_ml, (float*)out, out_stride, H, D, splits, gate, ldg));
   else
     DSP_REQUIRE(false, "dsp_attn_combine: unknown dtype %d", dtype);
   DSP_CHECK_LAUNCH("dsp_attn_combine");
   return 0;
+}
+
+extern "C" int dsp_attn_combine(const float* part_o, const float* part_ml, void* out, long out_stride,
+                                int num_tokens, int H, int D, int splits, int dtype,
+                                cudaStream_t stream) {
+  return dsp_attn_combine_gated(part_o, part_ml, out, out_stride, num_tokens, H, D, splits, dtype, nullptr, 0, stream);
 }

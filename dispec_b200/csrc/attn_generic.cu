@@ -13,7 +13,8 @@
 // exp(s_j) / (exp(z) + sum exp(s_j)), z = sink_values[head] (unscaled), or 0 without `sink_values`;
 // the running pair starts at (m, l) = (z, 1) instead of (-inf, 0).
 // With `turn_freq` (float [Dv/2]) the result of every head is turned back: pair (m, m + Dv/2) by
-// -p * turn_freq[m] (the values were stored turned by their own positions).  Any head_dim that is a multiple of 4 (float) / 8 (bfloat16) up to
+// -p * turn_freq[m] (the values were stored turned by their own positions).  With `gate` (float, row stride ldg, laid
+// out like the output's columns) every result is multiplied by the sigmoid of its gate value.  Any head_dim that is a multiple of 4 (float) / 8 (bfloat16) up to
 // 512, any G.  This kernel is the attention of the 32-bit path and the fallback of the
 // bfloat16 path for head sizes the tensor-core kernel is not built for.
 //
@@ -35,7 +36,7 @@ attn_generic_kernel(const T* __restrict__ q, long q_stride, const T* __restrict_
                     const int* __restrict__ seq_of_token, void* __restrict__ out, int out_dtype, long out_stride,
                     int H, int KVH, int D, int Dv, int page_size, int num_pages, int window, int mask_mode,
                     int keep_first, float scale, int sink, const float* __restrict__ sink_values,
-                    const float* __restrict__ turn_freq, int* err) {
+                    const float* __restrict__ turn_freq, const float* __restrict__ gate, long ldg, int* err) {
   extern __shared__ float smem[];
   float* qs = smem;                       // [GCHUNK][D]
   float* ps = qs + GCHUNK * D;            // [GCHUNK][THREADS]
@@ -162,10 +163,13 @@ attn_generic_kernel(const T* __restrict__ q, long q_stride, const T* __restrict_
       for (int dd = 0; dd < DPT; ++dd) {
         const int d = tid + dd * THREADS;
         if (d >= Dv) continue;
+        const size_t col = (size_t)(kvh * G + g0 + g) * Dv + d;
+        float y = acc[g][dd] * inv;
+        if (gate) y /= 1.f + expf(-gate[(size_t)t * ldg + col]);
         if (turn_freq)
-          os[g * Dv + d] = acc[g][dd] * inv;
+          os[g * Dv + d] = y;
         else
-          st_any(out, out_dtype, (size_t)t * out_stride + (size_t)(kvh * G + g0 + g) * Dv + d, acc[g][dd] * inv);
+          st_any(out, out_dtype, (size_t)t * out_stride + col, y);
       }
     }
     if (turn_freq) {
@@ -190,7 +194,7 @@ extern "C" int dsp_attn_generic(const void* q, long q_stride, const void* k_pool
                                 const int* positions, const int* seq_of_token, void* out,
                                 long out_stride, int T, int H, int KVH, int D, int Dv, int page_size,
                                 int num_pages, int window, int mask_mode, int keep_first, float scale,
-                                int sink, const float* sink_values, const float* turn_freq, int dtype, int out_dtype,
+                                int sink, const float* sink_values, const float* turn_freq, const float* gate, long ldg, int dtype, int out_dtype,
                                 cudaStream_t stream) {
   if (T == 0) return 0;
   DSP_REQUIRE(KVH > 0 && H % KVH == 0, "dsp_attn_generic: H=%d is not a multiple of KVH=%d", H, KVH);
@@ -200,6 +204,7 @@ extern "C" int dsp_attn_generic(const void* q, long q_stride, const void* k_pool
   DSP_REQUIRE(KVH <= 65535, "dsp_attn_generic: too many KV heads");
   DSP_REQUIRE(mask_mode == 0 || mask_mode == 1, "dsp_attn_generic: unknown mask mode %d", mask_mode);
   DSP_REQUIRE(keep_first >= 0, "dsp_attn_generic: keep_first=%d", keep_first);
+  DSP_REQUIRE(!gate || !turn_freq, "dsp_attn_generic: results are gated or turned back, not both");
   DSP_REQUIRE(!turn_freq || Dv % 2 == 0, "dsp_attn_generic: values of an odd width %d cannot be turned", Dv);
   int* err = dsp_device_error_ptr();
   DSP_REQUIRE(err != nullptr, "dsp_attn_generic: no device error word");
@@ -216,7 +221,7 @@ extern "C" int dsp_attn_generic(const void* q, long q_stride, const void* k_pool
     attn_generic_kernel<float><<<grid, THREADS, smem, stream>>>(
         (const float*)q, q_stride, (const float*)k_pool, (const float*)v_pool, page_table, pt_stride,
         positions, seq_of_token, out, out_dtype, out_stride, H, KVH, D, Dv, page_size, num_pages, window,
-        mask_mode, keep_first, scale, sink, sink_values, turn_freq, err);
+        mask_mode, keep_first, scale, sink, sink_values, turn_freq, gate, ldg, err);
   } else if (dtype == DSP_BF16) {
     static size_t configured = 0;
     if (smem > configured) {
@@ -227,7 +232,7 @@ extern "C" int dsp_attn_generic(const void* q, long q_stride, const void* k_pool
     attn_generic_kernel<bf16><<<grid, THREADS, smem, stream>>>(
         (const bf16*)q, q_stride, (const bf16*)k_pool, (const bf16*)v_pool, page_table, pt_stride,
         positions, seq_of_token, out, out_dtype, out_stride, H, KVH, D, Dv, page_size, num_pages, window,
-        mask_mode, keep_first, scale, sink, sink_values, turn_freq, err);
+        mask_mode, keep_first, scale, sink, sink_values, turn_freq, gate, ldg, err);
   } else {
     DSP_REQUIRE(false, "dsp_attn_generic: unknown dtype %d", dtype);
   }

@@ -4,7 +4,8 @@
 // `sink_values`, of the head's own unscaled score z: the running pair of the online softmax starts
 // at (max, sum) = (z, 1) instead of (-inf, 0)).  With `turn_freq` every head's result is turned
 // back, pair (m, m + DV/2) by -p * turn_freq[m] (values that were stored turned by their own
-// positions).  Compiled per pair of widths.
+// positions).  With `gate` (float rows laid out like the output's columns) every result is multiplied by the
+// sigmoid of its gate value (split results: where they are merged).  Compiled per pair of widths.
 //
 // A block of four warps takes one tile of the step's tile list and one key/value head: up to 64
 // query rows = (token, head of the group) pairs of one request, 16 rows a warp.  Keys come in
@@ -63,7 +64,7 @@ attn_sink_mma_kernel(const bf16* __restrict__ q, long ldq, const bf16* __restric
                      const int* __restrict__ tile_seq, const int* __restrict__ tile_tok0, void* __restrict__ out, int out_f32,
                      long ldo, int H, int G, int tpt, int page_size, int num_pages, int window, int mask_mode, int keep_first,
                      float scale_log2, int sink, const float* __restrict__ sink_values,
-                     const float* __restrict__ turn_freq, int tile_offset, int splits,
+                     const float* __restrict__ turn_freq, const float* __restrict__ gate, long ldg, int tile_offset, int splits,
                      float* __restrict__ part_o, float* __restrict__ part_ml, int* err) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* Qs = reinterpret_cast<bf16*>(smem_raw);  // [BM][LDK]
@@ -265,6 +266,14 @@ attn_sink_mma_kernel(const bf16* __restrict__ q, long ldq, const bf16* __restric
           o[i + DV / 16][2 * h + e] = v * cn - u * sn;
         }
     }
+    if (gate) {
+      const float* gr = gate + token * ldg + (size_t)head * DV + (lane & 3) * 2;
+#pragma unroll
+      for (int i = 0; i < DV / 8; ++i) {
+        o[i][2 * h] /= 1.f + expf(-gr[i * 8]);
+        o[i][2 * h + 1] /= 1.f + expf(-gr[i * 8 + 1]);
+      }
+    }
     if (out_f32) {  // 32-bit rows for a consumer that combines heads before it rounds
       float* dst = reinterpret_cast<float*>(out) + token * ldo + (size_t)head * DV + (lane & 3) * 2;
 #pragma unroll
@@ -287,11 +296,11 @@ extern "C" int DSP_CAT(dsp_attn_sink_mma_k, DSP_DK, _v, DSP_DV)(
     const void* q, long ldq, const void* k_pool, const void* v_pool, const int* page_table, int pt_stride,
     const int* q_start, const int* ctx_len, const int* tile_seq, const int* tile_tok0, int tile_offset, int num_tiles,
     void* out, int out_f32, long ldo, int H, int G, int tpt, int page_size, int num_pages, int window, int mask_mode, int keep_first,
-    float scale, int sink, const float* sink_values, const float* turn_freq, int splits, float* part_o, float* part_ml, int* err,
+    float scale, int sink, const float* sink_values, const float* turn_freq, const float* gate, long ldg, int splits, float* part_o, float* part_ml, int* err,
     cudaStream_t stream) {
   if (num_tiles == 0) return 0;
   if (G <= 0 || H % G || tpt <= 0 || tpt * (H / G) > BM || G > 65535 || page_size <= 0 || !err) return 2;
-  if (mask_mode < 0 || mask_mode > 1 || keep_first < 0) return 2;
+  if (mask_mode < 0 || mask_mode > 1 || keep_first < 0 || (gate && turn_freq)) return 2;
   if (splits < 1 || splits > 32 || (splits > 1 && (!part_o || !part_ml))) return 2;
   if (((uintptr_t)q % 16) || ((uintptr_t)k_pool % 16) || ((uintptr_t)v_pool % 16) || ((uintptr_t)out % (out_f32 ? 8 : 4)) || ldq % 8 || ldo % 2)
     return 3;
@@ -305,7 +314,7 @@ extern "C" int DSP_CAT(dsp_attn_sink_mma_k, DSP_DK, _v, DSP_DV)(
   const cudaError_t e = launch_plain(attn_sink_mma_kernel, dim3(num_tiles, G, splits), dim3(128), smem, stream, (const bf16*)q, ldq,
                                      (const bf16*)k_pool, (const bf16*)v_pool, page_table, pt_stride, q_start, ctx_len,
                                      tile_seq, tile_tok0, out, out_f32, ldo, H, G, tpt, page_size, num_pages, window,
-                                     mask_mode, keep_first, scale * 1.4426950408889634f, sink, sink_values, turn_freq, tile_offset,
+                                     mask_mode, keep_first, scale * 1.4426950408889634f, sink, sink_values, turn_freq, gate, ldg, tile_offset,
                                      splits, part_o, part_ml, err);
   return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? 0 : 1;
 }

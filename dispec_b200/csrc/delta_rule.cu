@@ -20,18 +20,18 @@
 // so that with x_j = v_j - gamma_j S0^T k_j both are fixed 8 x 8 matrices times x: u = P x, o = gamma S0^T q + N x.
 //   delta_prepare_kernel   forms P (rows already times D_8i) and N of every run and head, all runs in parallel
 //                          (`coef` [T, H, 20]: row i of P, row i of N, gamma_i, gamma_8, two spare).
-//   delta_runs_kernel      the sequential part: a block takes 16 value columns of one head and request and walks
-//                          its runs; the state stays in registers (a warp holds 32 state rows, SLICES lanes
+//   delta_runs_kernel      the sequential part: a block takes 8 value columns of one head and request and walks
+//                          its runs; the state stays in registers (a warp holds 32 state rows, eight lanes
 //                          share the rows of a column), the products S0^T k and S0^T q of eight tokens are added
-//                          over lanes together (each exchange halves what a lane still holds) and over warps
-//                          in shared memory; rows arrive by cp.async two runs ahead.
+//                          over lanes together (each exchange halves what a lane still holds; a lane counts the tokens
+//                          from its own, so that what it keeps always comes first) and over warps in shared memory; rows arrive by cp.async two runs ahead.
 // A request whose first row carries a negative position (a padding row of a captured step) is skipped: its
 // state slot belongs to someone else.
 #include "common.cuh"
 
 namespace {
 
-constexpr int RUN = 8, COEF = 20, COLS = 16;
+constexpr int RUN = 8, COEF = 20, SLICES = 8, COLS = 8;
 
 struct DeltaArgs {
   const float* rows;  // [T, ld]
@@ -176,12 +176,21 @@ delta_prepare_kernel(const DeltaArgs p, const int* __restrict__ run_seq, const i
   const int tid = threadIdx.x, ldm = (p.dim + 3) / 4 * 4 + 4;
   float* ks = smem;             // [RUN][ldm]
   float* qs = smem + RUN * ldm;
-  for (int idx = tid; idx < RUN * ldm; idx += 64) {
-    const int r = idx / ldm, i = idx % ldm;
-    const bool on = r < n && i < p.dim;
-    const float* row = p.rows + (size_t)(row0 + (on ? r : 0)) * p.ld + (size_t)group * p.dim + (on ? i : 0);
-    ks[idx] = on ? row[p.k_off] : 0.f;
-    qs[idx] = on ? row[p.q_off] : 0.f;
+  const bool wide = p.dim % 4 == 0 && p.ld % 4 == 0 && p.k_off % 4 == 0 && p.q_off % 4 == 0 && ((uintptr_t)p.rows & 15) == 0;
+#pragma unroll
+  for (int r = 0; r < RUN; ++r) {
+    const float* row = p.rows + (size_t)(row0 + min(r, n - 1)) * p.ld + (size_t)group * p.dim;
+    if (wide) {
+      for (int i = tid * 4; i < p.dim; i += 256) {
+        *reinterpret_cast<float4*>(ks + r * ldm + i) = r < n ? *reinterpret_cast<const float4*>(row + p.k_off + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        *reinterpret_cast<float4*>(qs + r * ldm + i) = r < n ? *reinterpret_cast<const float4*>(row + p.q_off + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+    } else {
+      for (int i = tid; i < ldm; i += 64) {
+        ks[r * ldm + i] = r < n && i < p.dim ? row[p.k_off + i] : 0.f;
+        qs[r * ldm + i] = r < n && i < p.dim ? row[p.q_off + i] : 0.f;
+      }
+    }
   }
   __syncthreads();
   {
@@ -291,12 +300,12 @@ struct Walk {
   static constexpr size_t smem = sizeof(float) * (stages * stage + meet + RUN * COLS * 2);
 };
 
-// PARTS warps of 32 state rows; SLICES lanes share the rows of a column, a lane holds 32 / SLICES rows of
-// SLICES / 2 columns
-template <int PARTS, int SLICES>
+// PARTS warps of 32 state rows; SLICES lanes share the rows of a column, a lane holds 32 / SLICES rows of two columns
+template <int PARTS>
 __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs p) {
   using L = Walk<PARTS>;
-  constexpr int ROWS = 32 / SLICES, NC = SLICES / 2, THREADS = 32 * PARTS, DP = L::rows;
+  constexpr int ROWS = 32 / SLICES, NC = 2, THREADS = 32 * PARTS, DP = L::rows;
+  static_assert(RUN == SLICES && COLS == NC * 32 / SLICES, "a lane ends with one token, a warp covers the block's columns");
   extern __shared__ __align__(16) float smem[];
   float* meet = smem + L::stages * L::stage;
   f32x2* us = reinterpret_cast<f32x2*>(meet + L::meet);  // [RUN][COLS]: (u, u)
@@ -336,14 +345,16 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
       for (int i = tid; i < (RUN - n) * COLS; i += THREADS) buf[2 * RUN * DP + n * COLS + i] = 0.f;
       for (int i = tid; i < (RUN - n) * COEF; i += THREADS) buf[2 * RUN * DP + RUN * COLS + n * COEF + i] = 0.f;
     }
+    static_assert(RUN * DP / 4 == 2 * THREADS, "two 16-byte pieces a thread and plane");
 #pragma unroll
     for (int pl = 0; pl < 2; ++pl) {
       const float* src = p.rows + (size_t)base * p.ld + (pl == 0 ? p.k_off : p.q_off) + (size_t)group * p.dim;
       float* dst = buf + pl * RUN * DP;
       if (wide) {
-        for (int idx = tid; idx < n * (DP / 4); idx += THREADS) {
-          const int r = idx / (DP / 4), i = idx % (DP / 4) * 4;
-          if (i < p.dim) cp_async16(dst + r * DP + i, src + (size_t)r * p.ld + i);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          const int r = tid / (DP / 4) + j * (RUN / 2), i = tid % (DP / 4) * 4;
+          if (r < n && i < p.dim) cp_async16(dst + r * DP + i, src + (size_t)r * p.ld + i);
         }
       } else {
         for (int idx = tid; idx < n * DP; idx += THREADS) {
@@ -355,9 +366,9 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
     float* vs = buf + 2 * RUN * DP;
     const float* vsrc = p.rows + (size_t)base * p.ld + p.v_off + (size_t)head * p.vdim + col0;
     if (v_wide) {
-      for (int idx = tid; idx < n * (COLS / 4); idx += THREADS) {
-        const int r = idx / (COLS / 4), i = idx % (COLS / 4) * 4;
-        if (col0 + i < p.vdim) cp_async16(vs + r * COLS + i, vsrc + (size_t)r * p.ld + i);
+      if (tid < RUN * COLS / 4) {
+        const int r = tid / (COLS / 4), i = tid % (COLS / 4) * 4;
+        if (r < n && col0 + i < p.vdim) cp_async16(vs + r * COLS + i, vsrc + (size_t)r * p.ld + i);
       }
     } else {
       for (int idx = tid; idx < n * COLS; idx += THREADS) {
@@ -366,8 +377,9 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
       }
     }
     float* cs = vs + RUN * COLS;
-    for (int idx = tid; idx < n * (COEF / 4); idx += THREADS)
-      cp_async16(cs + idx * 4, p.coef + ((size_t)(base + idx / (COEF / 4)) * p.H + head) * COEF + idx % (COEF / 4) * 4);
+#pragma unroll
+    for (int idx = THREADS - 1 - tid; idx < RUN * (COEF / 4); idx += THREADS)  // (from the other end: the first threads have the values)
+      if (idx < n * (COEF / 4)) cp_async16(cs + idx * 4, p.coef + ((size_t)(base + idx / (COEF / 4)) * p.H + head) * COEF + idx % (COEF / 4) * 4);
   };
 
 #pragma unroll
@@ -378,6 +390,10 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
   asm volatile("cp.async.wait_group 1;\n");
   __syncthreads();
 
+  int mine[RUN];  // where this lane's rows of token t ^ slice lie in a stage
+#pragma unroll
+  for (int t = 0; t < RUN; ++t) mine[t] = (t ^ slice) * DP + row0;
+
   int turn = 0;
   for (int base = t0; base < t1; base += RUN, turn = (turn + 1) & 3) {
     const float* buf = smem + turn * L::stage;
@@ -385,20 +401,24 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
     if (base + 2 * RUN < t1) stage_run(base + 2 * RUN, smem + ((turn + 2) & 3) * L::stage);
     asm volatile("cp.async.commit_group;\n");
 
-    // S0^T k and S0^T q of the run's tokens over this lane's rows: value (token * 2 + which) * NC + column
+    // S0^T k and S0^T q of the run's tokens over this lane's rows; t counts from this lane's token: value
+    // (t * 2 + which) * NC + column belongs to token t ^ slice
+    static_assert(ROWS == 4, "a lane's rows are one 16-byte piece");
     float acc[RUN * 2 * NC];
+    ulonglong2 kr[RUN], qr[RUN];  // the keys stay for the update of the state
+#pragma unroll
+    for (int t = 0; t < RUN; ++t) {
+      kr[t] = *reinterpret_cast<const ulonglong2*>(buf + mine[t]);
+      qr[t] = *reinterpret_cast<const ulonglong2*>(buf + RUN * DP + mine[t]);
+    }
 #pragma unroll
     for (int t = 0; t < RUN; ++t)
 #pragma unroll
       for (int w = 0; w < 2; ++w) {
-        const f32x2* x = reinterpret_cast<const f32x2*>(buf + (w * RUN + t) * DP + row0);
+        const ulonglong2 x = w == 0 ? kr[t] : qr[t];
         f32x2 s[NC];
 #pragma unroll
-        for (int k = 0; k < ROWS / 2; ++k) {
-          const f32x2 xk = x[k];
-#pragma unroll
-          for (int c = 0; c < NC; ++c) s[c] = k == 0 ? mul2(S[k][c], xk) : fma2(S[k][c], xk, s[c]);
-        }
+        for (int c = 0; c < NC; ++c) s[c] = fma2(S[1][c], x.y, mul2(S[0][c], x.x));
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
           float a, b;
@@ -406,27 +426,18 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
           acc[(t * 2 + w) * NC + c] = a + b;
         }
       }
-    // sums over the slices: each exchange leaves a lane half of its values, eight at the end
+    // sums over the slices: each exchange leaves a lane the first half of its values (the tokens nearer to its own, whose
+    // partner's are in that partner's second half), at the end those of token `slice`
 #pragma unroll
     for (int o = SLICES / 2, m = RUN * NC; o > 0; o >>= 1, m >>= 1) {
-      const bool upper = (slice & o) != 0;
 #pragma unroll
       for (int i = 0; i < RUN * NC; ++i)
-        if (i < m) {
-          const float keep = upper ? acc[i + m] : acc[i], give = upper ? acc[i] : acc[i + m];
-          acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
-        }
+        if (i < m) acc[i] += __shfl_xor_sync(0xffffffffu, acc[i + m], o);
     }
     {
-      float* dst = meet + part * RUN * L::token;
-      constexpr int TPL = RUN / SLICES;  // tokens a lane ends with
-      static_assert(TPL * 2 * NC == 8, "a lane ends with eight values");
-#pragma unroll
-      for (int e = 0; e < TPL * 2; ++e)
-#pragma unroll
-        for (int c = 0; c < NC; c += 2)
-          *reinterpret_cast<float2*>(dst + (slice * TPL + e / 2) * L::token + (e & 1) * COLS + cl + c) =
-              make_float2(acc[e * NC + c], acc[e * NC + c + 1]);
+      float* dst = meet + (part * RUN + slice) * L::token + cl;
+      *reinterpret_cast<float2*>(dst) = make_float2(acc[0], acc[1]);
+      *reinterpret_cast<float2*>(dst + COLS) = make_float2(acc[2], acc[3]);
     }
     __syncthreads();
     // u and o: a thread a (token, column), the eight tokens of a column in neighbouring lanes
@@ -451,13 +462,17 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
       }
       const float gamma = cf[2 * RUN], x = vs[t * COLS + c] - gamma * r;
       o *= gamma;
-      float u = 0.f;
+      float u = 0.f, u2 = 0.f, o2 = 0.f;
 #pragma unroll
-      for (int j = 0; j < RUN; ++j) {
-        const float xj = __shfl_sync(0xffffffffu, x, j, RUN);
+      for (int j = 0; j < RUN; j += 2) {
+        const float xj = __shfl_sync(0xffffffffu, x, j, RUN), xk = __shfl_sync(0xffffffffu, x, j + 1, RUN);
         u = fmaf(P[j], xj, u);
         o = fmaf(N[j], xj, o);
+        u2 = fmaf(P[j + 1], xk, u2);
+        o2 = fmaf(N[j + 1], xk, o2);
       }
+      u += u2;
+      o += o2;
       us[t * COLS + c] = pack2f(u, u);
       if (base + t < t1 && col0 + c < p.vdim) p.out[(size_t)(base + t) * p.ldo + (size_t)head * p.vdim + col0 + c] = o;
     }
@@ -469,18 +484,15 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
     for (int k = 0; k < ROWS / 2; ++k)
 #pragma unroll
       for (int c = 0; c < NC; ++c) S[k][c] = mul2(g2, S[k][c]);
+    ulonglong2 u[RUN];  // both columns' (u, u) of token t ^ slice
+#pragma unroll
+    for (int t = 0; t < RUN; ++t) u[t] = *reinterpret_cast<const ulonglong2*>(us + (t ^ slice) * COLS + cl);
 #pragma unroll
     for (int t = 0; t < RUN; ++t) {
-      const f32x2* x = reinterpret_cast<const f32x2*>(buf + t * DP + row0);
-      f32x2 u[NC];
-#pragma unroll
-      for (int c = 0; c < NC; ++c) u[c] = us[t * COLS + cl + c];
-#pragma unroll
-      for (int k = 0; k < ROWS / 2; ++k) {
-        const f32x2 xk = x[k];
-#pragma unroll
-        for (int c = 0; c < NC; ++c) S[k][c] = fma2(xk, u[c], S[k][c]);
-      }
+      S[0][0] = fma2(kr[t].x, u[t].x, S[0][0]);
+      S[0][1] = fma2(kr[t].x, u[t].y, S[0][1]);
+      S[1][0] = fma2(kr[t].y, u[t].x, S[1][0]);
+      S[1][1] = fma2(kr[t].y, u[t].y, S[1][1]);
     }
   }
   asm volatile("cp.async.wait_group 0;\n");
@@ -506,14 +518,13 @@ int launch_single(const DeltaArgs& a, int S, cudaStream_t stream) {
 
 template <int PARTS>
 int launch_runs(const DeltaArgs& a, int S, cudaStream_t stream) {
-  constexpr int SLICES = 8;
   static bool configured = false;
   if (!configured) {
-    DSP_CUDA(cudaFuncSetAttribute(delta_runs_kernel<PARTS, SLICES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Walk<PARTS>::smem));
+    DSP_CUDA(cudaFuncSetAttribute(delta_runs_kernel<PARTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Walk<PARTS>::smem));
     configured = true;
   }
   const dim3 grid((a.vdim + COLS - 1) / COLS, a.H, S);
-  DSP_CUDA(launch_plain(delta_runs_kernel<PARTS, SLICES>, grid, dim3(32 * PARTS), Walk<PARTS>::smem, stream, a));
+  DSP_CUDA(launch_plain(delta_runs_kernel<PARTS>, grid, dim3(32 * PARTS), Walk<PARTS>::smem, stream, a));
   DSP_CHECK_LAUNCH("dsp_delta_rule");
   return 0;
 }

@@ -17,7 +17,7 @@
 //                              the first two kinds of heads divided by their length, x / sqrt(sum(x^2) + eps), the
 //                              first one then times a factor; and, for a delta rule, per token and head
 //                              sigmoid(raw b) and -exp(A_log) * softplus(raw a + bias) as `steps` [T, 2, H].  A warp takes
-//                              one head of one token.
+//                              one head of one token, or of four neighbouring ones in steps with portions of prompts.
 //
 // Every token has a block (or a row of blocks) of its own: its taps come from the rows of the step, and,
 // before the first token the step brings for the request, from the state slot.  The block of that
@@ -236,25 +236,13 @@ qkv_conv_rotate_store_kernel(const ConvIn p, const int* __restrict__ page_table,
     for (int c = tid; c < p.channels; c += blockDim.x) keep_inputs(p, r, hist, c);
 }
 
-// One warp a (token, head); blockIdx.y counts the heads, the last one stands for the steps.
+// One warp a (token or TOK tokens, head); blockIdx.y counts the heads, the last one stands for the steps.
 constexpr int HEAD_WARPS = 8, HEAD_QUADS = 2;  // HEAD_QUADS: groups of four channels a lane keeps in registers
 
-__global__ void __launch_bounds__(32 * HEAD_WARPS)
-conv_heads_kernel(const ConvIn p, int T, int A, int B, int dim, int vdim, float eps, float a_scale, float* __restrict__ out,
-                  long ldo, int b_off, int a_off, int H, const float* __restrict__ step_bias,
-                  const float* __restrict__ a_log, float* __restrict__ steps) {
-  const int t = blockIdx.x * HEAD_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31, head = blockIdx.y;
-  if (t >= T || p.positions[t] < 0) return;
-  if (head == A + B + H) {
-    for (int h = lane; h < H; h += 32) {
-      steps[(size_t)t * 2 * H + h] = 1.f / (1.f + expf(-ld_any(p.u, p.dtype, (size_t)t * p.ld + b_off + h)));
-      steps[((size_t)t * 2 + 1) * H + h] = -expf(a_log[h]) * softplus_f(ld_any(p.u, p.dtype, (size_t)t * p.ld + a_off + h) + step_bias[h]);
-    }
-    return;
-  }
-  const bool unit = head < A + B;
-  const int c0 = unit ? head * dim : (A + B) * dim + (head - A - B) * vdim, n = unit ? dim : vdim;
-  const float factor = head < A ? a_scale : 1.f;
+// one token: c0, n: the head's columns
+__device__ __forceinline__ void conv_head_token(const ConvIn& p, int t, int lane, int c0, int n, bool unit, float factor, float eps,
+                                                float* __restrict__ out, long ldo) {
+  if (p.positions[t] < 0) return;
   const Turn r = turn_of(p, t);
   if (r.count == 0) return;
   float* hist = p.taps > 1 ? p.hist + (size_t)p.state_slot[r.seq] * (p.taps - 1) * p.channels : nullptr;
@@ -295,6 +283,82 @@ conv_heads_kernel(const ConvIn p, int T, int A, int B, int dim, int vdim, float 
   }
   if (r.owner && p.taps > 1)
     for (int c = lane; c < n; c += 32) keep_inputs(p, r, hist, c0 + c);
+}
+
+// TOK neighbouring tokens of one request whose taps all lie in the step's rows: a row is loaded once for all of them,
+// the weights once (the same sums in the same order)
+template <int TAPS, int TOK>
+__device__ __forceinline__ void conv_head_run(const ConvIn& p, int t, int lane, int c0, int n, bool unit, float factor, float eps,
+                                              float* __restrict__ out, long ldo) {
+  float4 y[TOK][HEAD_QUADS];
+  float ss[TOK] = {};
+  auto silu = [](float v) { return v / (1.f + expf(-v)); };
+#pragma unroll
+  for (int k = 0; k < HEAD_QUADS; ++k) {
+    const int i = (lane + 32 * k) * 4;
+    if (i >= n) break;
+    const float* u = reinterpret_cast<const float*>(p.u) + (size_t)(t - (TAPS - 1)) * p.ld + c0 + i;
+    float4 x[TOK + TAPS - 1], w[TAPS];
+#pragma unroll
+    for (int j = 0; j < TOK + TAPS - 1; ++j) x[j] = *reinterpret_cast<const float4*>(u + (size_t)j * p.ld);
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j] = *reinterpret_cast<const float4*>(p.w + (size_t)j * p.channels + c0 + i);
+#pragma unroll
+    for (int m = 0; m < TOK; ++m) {
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        a.x = fmaf(w[j].x, x[m + j].x, a.x);
+        a.y = fmaf(w[j].y, x[m + j].y, a.y);
+        a.z = fmaf(w[j].z, x[m + j].z, a.z);
+        a.w = fmaf(w[j].w, x[m + j].w, a.w);
+      }
+      y[m][k] = make_float4(silu(a.x), silu(a.y), silu(a.z), silu(a.w));
+      ss[m] += (y[m][k].x * y[m][k].x + y[m][k].y * y[m][k].y) + (y[m][k].z * y[m][k].z + y[m][k].w * y[m][k].w);
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < TOK; ++m) {
+    const float f = unit ? factor / sqrtf(warp_sum(ss[m]) + eps) : 1.f;
+#pragma unroll
+    for (int k = 0; k < HEAD_QUADS; ++k) {
+      const int i = (lane + 32 * k) * 4;
+      if (i < n) *reinterpret_cast<float4*>(out + (size_t)(t + m) * ldo + c0 + i) = make_float4(y[m][k].x * f, y[m][k].y * f, y[m][k].z * f, y[m][k].w * f);
+    }
+  }
+}
+
+template <int TOK>
+__global__ void __launch_bounds__(32 * HEAD_WARPS)
+conv_heads_kernel(const ConvIn p, int T, int A, int B, int dim, int vdim, float eps, float a_scale, float* __restrict__ out,
+                  long ldo, int b_off, int a_off, int H, const float* __restrict__ step_bias,
+                  const float* __restrict__ a_log, float* __restrict__ steps) {
+  const int t = (blockIdx.x * HEAD_WARPS + (threadIdx.x >> 5)) * TOK, lane = threadIdx.x & 31, head = blockIdx.y;
+  if (t >= T) return;
+  const int end = min(T, t + TOK);
+  if (head == A + B + H) {
+    for (int idx = lane; idx < (end - t) * H; idx += 32) {
+      const int tok = t + idx / H, h = idx % H;
+      if (p.positions[tok] < 0) continue;
+      steps[(size_t)tok * 2 * H + h] = 1.f / (1.f + expf(-ld_any(p.u, p.dtype, (size_t)tok * p.ld + b_off + h)));
+      steps[((size_t)tok * 2 + 1) * H + h] = -expf(a_log[h]) * softplus_f(ld_any(p.u, p.dtype, (size_t)tok * p.ld + a_off + h) + step_bias[h]);
+    }
+    return;
+  }
+  const bool unit = head < A + B;
+  const int c0 = unit ? head * dim : (A + B) * dim + (head - A - B) * vdim, n = unit ? dim : vdim;
+  const float factor = head < A ? a_scale : 1.f;
+  if (TOK > 1 && end == t + TOK && p.taps >= 2 && p.taps <= 4 && n % 4 == 0 && c0 % 4 == 0 && n <= 128 * HEAD_QUADS && in_fours(p) &&
+      ldo % 4 == 0 && ((uintptr_t)out & 15) == 0) {
+    const int seq = p.seq_of_token[t];
+    if (p.positions[t] >= 0 && p.seq_of_token[end - 1] == seq && t - p.q_start[seq] >= p.taps - 1) {
+      if (p.taps == 4) conv_head_run<4, TOK>(p, t, lane, c0, n, unit, factor, eps, out, ldo);
+      else if (p.taps == 3) conv_head_run<3, TOK>(p, t, lane, c0, n, unit, factor, eps, out, ldo);
+      else conv_head_run<2, TOK>(p, t, lane, c0, n, unit, factor, eps, out, ldo);
+      return;
+    }
+  }
+  for (int tok = t; tok < end; ++tok) conv_head_token(p, tok, lane, c0, n, unit, factor, eps, out, ldo);
 }
 
 int check(const ConvIn& p, const char* name) {
@@ -359,8 +423,10 @@ extern "C" int dsp_conv_heads(const void* u, int dtype, long ld, int taps, const
   if (const int rc = check(p, "dsp_conv_heads")) return rc;
   DSP_REQUIRE(out && w && step_bias && a_log && steps, "dsp_conv_heads: missing operand");
   DSP_REQUIRE(A + B + H + 1 <= 65535, "dsp_conv_heads: too many heads");
-  DSP_CUDA(launch_plain(conv_heads_kernel, dim3((T + HEAD_WARPS - 1) / HEAD_WARPS, A + B + H + 1), dim3(32 * HEAD_WARPS), 0, stream,
-                        p, T, A, B, dim, vdim, eps, a_scale, out, ldo, b_off, a_off, H, step_bias, a_log, steps));
+  const int tok = T >= 256 ? 4 : 1, per = HEAD_WARPS * tok;
+  DSP_CUDA(launch_plain(tok == 4 ? conv_heads_kernel<4> : conv_heads_kernel<1>, dim3((T + per - 1) / per, A + B + H + 1),
+                        dim3(32 * HEAD_WARPS), 0, stream, p, T, A, B, dim, vdim, eps, a_scale, out, ldo, b_off, a_off, H, step_bias,
+                        a_log, steps));
   DSP_CHECK_LAUNCH("dsp_conv_heads");
   return 0;
 }

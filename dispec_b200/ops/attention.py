@@ -37,7 +37,8 @@ def paged_attention_generic(q: torch.Tensor, q_stride: int, k_pool: torch.Tensor
                             seq_of_token: torch.Tensor, out: torch.Tensor, num_heads: int,
                             num_kv_heads: int, head_dim: int, window: int, scale: float,
                             sink: bool = False, chunked: bool = False, sink_values: torch.Tensor | None = None,
-                            turn_freq: torch.Tensor | None = None, keep_first: int = 0) -> torch.Tensor:
+                            turn_freq: torch.Tensor | None = None, keep_first: int = 0,
+                            gate: torch.Tensor | None = None) -> torch.Tensor:
     """32-bit arithmetic kernel, any value size up to 512 and any group size.
 
     q: element (t, h, d) at q.data_ptr + (t * q_stride + h * D + d); out: [T, H * Dv], Dv being the
@@ -48,7 +49,8 @@ def paged_attention_generic(q: torch.Tensor, q_stride: int, k_pool: torch.Tensor
     0..F-1.  ``sink``: the softmax has one more key
     of score 0 and no value (weights exp(s_j) / (1 + sum exp(s_j))); with ``sink_values`` (float32
     [H]) that key's score is the head's own number, unscaled.  ``turn_freq`` (float32 [Dv/2]):
-    every head's result is turned back, pair (m, m + Dv/2) by -p * turn_freq[m].
+    every head's result is turned back, pair (m, m + Dv/2) by -p * turn_freq[m].  ``gate`` (float32, shaped like
+    ``out``): every result is multiplied by the sigmoid of its gate value.
     """
     assert q.is_cuda and k_pool.is_cuda, "CUDA tensors only (there is no CPU path)"
     T = positions.shape[0]
@@ -60,13 +62,20 @@ def paged_attention_generic(q: torch.Tensor, q_stride: int, k_pool: torch.Tensor
     assert page_table.dtype == torch.int32 and page_table.stride(1) == 1
     assert positions.dtype == torch.int32 and seq_of_token.dtype == torch.int32
     _check_sink_turn(sink, sink_values, turn_freq, num_heads, dv)
+    _check_gate(gate, out, turn_freq)
     L.check(L.core().dsp_attn_generic(
         L.ptr(q), L.i64(q_stride), L.ptr(k_pool), L.ptr(v_pool), L.ptr(page_table),
         page_table.stride(0), L.ptr(positions), L.ptr(seq_of_token), L.ptr(out),
         L.i64(out.stride(0)), T, num_heads, num_kv_heads, head_dim, dv, page_size, num_pages,
         window, int(bool(chunked) and window > 0), int(keep_first), L.f32(scale), int(bool(sink)), L.ptr(sink_values),
-        L.ptr(turn_freq), L.dtype_code(q.dtype), L.dtype_code(out.dtype), L.stream_handle()))
+        L.ptr(turn_freq), L.ptr(gate), L.i64(gate.stride(0) if gate is not None else 0), L.dtype_code(q.dtype),
+        L.dtype_code(out.dtype), L.stream_handle()))
     return out
+
+
+def _check_gate(gate, out, turn_freq) -> None:
+    assert gate is None or (turn_freq is None and gate.is_cuda and gate.dtype == torch.float32 and gate.shape == out.shape
+                            and gate.stride(1) == 1)
 
 
 def _check_sink_turn(sink, sink_values, turn_freq, num_heads: int, value_dim: int) -> None:
@@ -404,11 +413,11 @@ def sink_attention_tiles(q, k_pool, v_pool, page_table, q_start, ctx_len, tile_s
                          num_heads, num_kv_heads, window, scale, sink, num_single: int = 0, splits: int = 1,
                          chunked: bool = False, sink_values: torch.Tensor | None = None,
                          turn_freq: torch.Tensor | None = None, positions: torch.Tensor | None = None,
-                         keep_first: int = 0) -> torch.Tensor:
+                         keep_first: int = 0, gate: torch.Tensor | None = None) -> torch.Tensor:
     """The tensor-core kernel over a tile list (``tokens per tile`` = 64 // group).  The first
     ``num_single`` tiles are single tokens (the first rows of the batch): with ``splits`` > 1
     their keys are cut into that many shares, merged by the combine kernel.  ``chunked``,
-    ``sink_values``, ``turn_freq``, ``keep_first``: as in ``paged_attention_generic``; ``positions`` (of the step's
+    ``sink_values``, ``turn_freq``, ``keep_first``, ``gate``: as in ``paged_attention_generic``; ``positions`` (of the step's
     tokens) is needed where split results are turned back."""
     num_pages, G, page_size, dk = k_pool.shape
     dv = v_pool.shape[3]
@@ -417,13 +426,15 @@ def sink_attention_tiles(q, k_pool, v_pool, page_table, q_start, ctx_len, tile_s
     fn = getattr(L.sink_attention_library(dk, dv), f"dsp_attn_sink_mma_k{dk}_v{dv}")
     tpt = SINK_ROWS_PER_TILE // (num_heads // num_kv_heads)
     _check_sink_turn(sink, sink_values, turn_freq, num_heads, dv)
+    _check_gate(gate, out, turn_freq)
+    ldg = L.i64(gate.stride(0) if gate is not None else 0)
     mask_mode = int(bool(chunked) and window > 0)
 
     def launch(offset, count, n_splits, part_o, part_ml):
         rc = fn(L.ptr(q), L.i64(q.stride(0)), L.ptr(k_pool), L.ptr(v_pool), L.ptr(page_table), page_table.stride(0),
                 L.ptr(q_start), L.ptr(ctx_len), L.ptr(tile_seq), L.ptr(tile_tok0), offset, count, L.ptr(out),
                 int(out.dtype == torch.float32), L.i64(out.stride(0)), num_heads, num_kv_heads, tpt, page_size, num_pages, window, mask_mode,
-                int(keep_first), L.f32(scale), int(bool(sink)), L.ptr(sink_values), L.ptr(turn_freq), n_splits, L.ptr(part_o), L.ptr(part_ml), ctypes.c_void_p(_device_error_address(q.device)),
+                int(keep_first), L.f32(scale), int(bool(sink)), L.ptr(sink_values), L.ptr(turn_freq), L.ptr(gate), ldg, n_splits, L.ptr(part_o), L.ptr(part_ml), ctypes.c_void_p(_device_error_address(q.device)),
                 L.stream_handle())
         L.LaunchCounter.n += 1
         if rc != 0:
@@ -439,9 +450,9 @@ def sink_attention_tiles(q, k_pool, v_pool, page_table, q_start, ctx_len, tile_s
                 L.ptr(part_o), L.ptr(part_ml), L.ptr(out), L.dtype_code(out.dtype), L.i64(out.stride(0)),
                 L.ptr(positions), L.ptr(turn_freq), num_single, num_heads, dv, splits, L.stream_handle()))
         else:
-            L.check(L.core().dsp_attn_combine(L.ptr(part_o), L.ptr(part_ml), L.ptr(out), L.i64(out.stride(0)),
-                                              num_single, num_heads, dv, splits, L.dtype_code(out.dtype),
-                                              L.stream_handle()))
+            L.check(L.core().dsp_attn_combine_gated(L.ptr(part_o), L.ptr(part_ml), L.ptr(out), L.i64(out.stride(0)),
+                                                    num_single, num_heads, dv, splits, L.dtype_code(out.dtype),
+                                                    L.ptr(gate), ldg, L.stream_handle()))
         first = num_single
     if num_tiles > first:
         launch(first, num_tiles - first, 1, None, None)
@@ -451,7 +462,7 @@ def sink_attention_tiles(q, k_pool, v_pool, page_table, q_start, ctx_len, tile_s
 def sink_paged_attention(ctx, q: torch.Tensor, cache, out: torch.Tensor, num_heads: int, num_kv_heads: int,
                          key_dim: int, value_dim: int, window: int, scale: float, sink: bool, chunked: bool = False,
                          sink_values: torch.Tensor | None = None, turn_freq: torch.Tensor | None = None,
-                         keep_first: int = 0) -> torch.Tensor:
+                         keep_first: int = 0, gate: torch.Tensor | None = None) -> torch.Tensor:
     """Attention of the step over pools whose keys and values have widths of their own, with an
     optional sink in the softmax: q [T, H * Dk] (already turned), out [T, H * Dv] (of q's type, or
     float32 for a consumer that combines heads before it rounds).  bfloat16 runs
@@ -459,7 +470,7 @@ def sink_paged_attention(ctx, q: torch.Tensor, cache, out: torch.Tensor, num_hea
     everything else (and float32 always) on the 32-bit kernel.  ``chunked``: ``window`` is the
     size of the chunks a position's keys come from; ``sink_values``: the sink's score per head;
     ``turn_freq``: results are turned back by the query's position; ``keep_first``: so many first keys
-    stay visible beside the window (``paged_attention_generic``)."""
+    stay visible beside the window; ``gate``: an output gate per element (``paged_attention_generic``)."""
     group = num_heads // num_kv_heads
     tpt = sink_tokens_per_tile(group, key_dim, value_dim)
     if q.dtype == torch.bfloat16 and tpt is not None and tpt in ctx.attention_tiles:
@@ -470,8 +481,8 @@ def sink_paged_attention(ctx, q: torch.Tensor, cache, out: torch.Tensor, num_hea
                                     tile_seq, tile_tok0, num_tiles, out, num_heads, num_kv_heads, window, scale, sink,
                                     num_single=ctx.num_decode_seqs, splits=splits, chunked=chunked,
                                     sink_values=sink_values, turn_freq=turn_freq, positions=ctx.positions,
-                                    keep_first=keep_first)
+                                    keep_first=keep_first, gate=gate)
     return paged_attention_generic(q, q.stride(0), cache.key_pool, cache.value_pool, cache.page_table,
                                    ctx.positions, ctx.seq_of_token, out, num_heads, num_kv_heads, key_dim,
                                    window, scale, sink=sink, chunked=chunked, sink_values=sink_values,
-                                   turn_freq=turn_freq, keep_first=keep_first)
+                                   turn_freq=turn_freq, keep_first=keep_first, gate=gate)

@@ -178,6 +178,8 @@ class SinkAttention(JoinableMixer):
         self.value_theta = float(value_theta) if value_theta is not None else None
         self.position_encoding = position_encoding
         self.value_mix = tuple(value_mix) if value_mix is not None else None
+        if out_gate and value_theta is not None:
+            raise ValueError("sink_attention: results are gated or turned back, not both")
         self.bias, self.values, self.out_gate = bool(bias), values, bool(out_gate)
         self.out_columns = num_heads * value_dim
         self.qkv_columns = (num_heads + num_kv_heads) * key_dim + (num_kv_heads * value_dim if values == "own" else 0)
@@ -250,14 +252,10 @@ class SinkAttention(JoinableMixer):
                                       ctx.dtype, v_other=v_other, blend=self.blend, q_norm=self.q_norm,
                                       k_norm=self.k_norm, norm_eps=self.norm_eps, v_norm=self.value_norm,
                                       v_inv_freq=self.value_freq, v_from_k=self.values == "keys")
-        # a gate reads the heads in 32-bit
-        o = torch.empty((q.shape[0], H * dv), dtype=torch.float32, device=q.device) if self.out_gate else out
-        attn_ops.sink_paged_attention(ctx, q, cache, o, H, G, dk, dv, self.window,
+        attn_ops.sink_paged_attention(ctx, q, cache, out, H, G, dk, dv, self.window,
                                       self.scale * self.position_encoding.score_scale(), bool(self.sink),
                                       chunked=self.mask == "chunk", sink_values=self.sink_values,
-                                      turn_freq=self.value_freq)
-        if self.out_gate:
-            norm32_ops.sigmoid_gate(o, z[:, self.qkv_columns:], out.dtype, out=out)
+                                      turn_freq=self.value_freq, gate=z[:, self.qkv_columns:] if self.out_gate else None)
 
 
 @register_part("mixer", "differential_attention")
