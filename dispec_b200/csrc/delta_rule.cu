@@ -297,7 +297,7 @@ struct Walk {
   static constexpr int stages = 4;
   static constexpr int token = 2 * COLS + 4;                                     // a token's S^T k and S^T q of the block's columns
   static constexpr int meet = PARTS * RUN * token;
-  static constexpr size_t smem = sizeof(float) * (stages * stage + meet + RUN * COLS * 2);
+  static constexpr size_t smem = sizeof(float) * (stages * stage + meet + RUN * COLS);
 };
 
 // PARTS warps of 32 state rows; SLICES lanes share the rows of a column, a lane holds 32 / SLICES rows of two columns
@@ -308,12 +308,15 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
   static_assert(RUN == SLICES && COLS == NC * 32 / SLICES, "a lane ends with one token, a warp covers the block's columns");
   extern __shared__ __align__(16) float smem[];
   float* meet = smem + L::stages * L::stage;
-  f32x2* us = reinterpret_cast<f32x2*>(meet + L::meet);  // [RUN][COLS]: (u, u)
+  float* us = meet + L::meet;  // [RUN][COLS]
   const int seq = p.first_seq + blockIdx.z, head = blockIdx.y, group = head / (p.H / p.G);
   const int t0 = p.q_start[seq], t1 = p.q_start[seq + 1];
   if (t1 <= t0 || p.positions[t0] < 0) return;
   const int tid = threadIdx.x, lane = tid & 31, part = tid >> 5;
-  const int slice = lane % SLICES, cl = lane / SLICES * NC;  // this lane's first column within the block's
+  // neighbouring lanes share rows (loads of 16 bytes at one address by neighbours cost half of what they cost spread
+  // over the warp), cl: this lane's first column within the block's
+  constexpr int GROUPS = 32 / SLICES;
+  const int slice = lane / GROUPS, cl = lane % GROUPS * NC;
   const int row0 = part * 32 + slice * ROWS, col0 = blockIdx.x * COLS;
   float* sp = p.state + ((size_t)p.state_slot[seq] * p.H + head) * p.dim * p.vdim;
 
@@ -335,6 +338,13 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
   for (int i = tid; i < L::stages * L::stage; i += THREADS) smem[i] = 0.f;
   __syncthreads();
 
+  // this thread's pieces of a run: where the first two lie in the rows, and the coefficients'
+  const int piece_r = tid / (DP / 4), piece_i = tid % (DP / 4) * 4;
+  const bool piece_on = wide && piece_i < p.dim;
+  const float* row_piece = p.rows + (size_t)piece_r * p.ld + (size_t)group * p.dim + piece_i;
+  const int val_r = tid / (COLS / 4), val_i = tid % (COLS / 4) * 4;
+  const bool val_on = v_wide && tid < RUN * COLS / 4 && col0 + val_i < p.vdim;
+  const float* val_piece = p.rows + (size_t)val_r * p.ld + p.v_off + (size_t)head * p.vdim + col0 + val_i;
   auto stage_run = [&](int base, float* buf) {
     const int n = min(RUN, t1 - base);
     if (n < RUN) {  // the last run: its missing tokens are rows of zeros
@@ -348,15 +358,13 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
     static_assert(RUN * DP / 4 == 2 * THREADS, "two 16-byte pieces a thread and plane");
 #pragma unroll
     for (int pl = 0; pl < 2; ++pl) {
-      const float* src = p.rows + (size_t)base * p.ld + (pl == 0 ? p.k_off : p.q_off) + (size_t)group * p.dim;
       float* dst = buf + pl * RUN * DP;
       if (wide) {
-#pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          const int r = tid / (DP / 4) + j * (RUN / 2), i = tid % (DP / 4) * 4;
-          if (r < n && i < p.dim) cp_async16(dst + r * DP + i, src + (size_t)r * p.ld + i);
-        }
+        const float* src = row_piece + (size_t)base * p.ld + (pl == 0 ? p.k_off : p.q_off);
+        if (piece_on && piece_r < n) cp_async16(dst + piece_r * DP + piece_i, src);
+        if (piece_on && piece_r + RUN / 2 < n) cp_async16(dst + (piece_r + RUN / 2) * DP + piece_i, src + RUN / 2 * p.ld);
       } else {
+        const float* src = p.rows + (size_t)base * p.ld + (pl == 0 ? p.k_off : p.q_off) + (size_t)group * p.dim;
         for (int idx = tid; idx < n * DP; idx += THREADS) {
           const int r = idx / DP, i = idx % DP;
           if (i < p.dim) cp_async4(dst + r * DP + i, src + (size_t)r * p.ld + i);
@@ -364,13 +372,10 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
       }
     }
     float* vs = buf + 2 * RUN * DP;
-    const float* vsrc = p.rows + (size_t)base * p.ld + p.v_off + (size_t)head * p.vdim + col0;
     if (v_wide) {
-      if (tid < RUN * COLS / 4) {
-        const int r = tid / (COLS / 4), i = tid % (COLS / 4) * 4;
-        if (r < n && col0 + i < p.vdim) cp_async16(vs + r * COLS + i, vsrc + (size_t)r * p.ld + i);
-      }
+      if (val_on && val_r < n) cp_async16(vs + val_r * COLS + val_i, val_piece + (size_t)base * p.ld);
     } else {
+      const float* vsrc = p.rows + (size_t)base * p.ld + p.v_off + (size_t)head * p.vdim + col0;
       for (int idx = tid; idx < n * COLS; idx += THREADS) {
         const int r = idx / COLS, i = idx % COLS;
         if (col0 + i < p.vdim) cp_async4(vs + idx, vsrc + (size_t)r * p.ld + i);
@@ -432,7 +437,7 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
     for (int o = SLICES / 2, m = RUN * NC; o > 0; o >>= 1, m >>= 1) {
 #pragma unroll
       for (int i = 0; i < RUN * NC; ++i)
-        if (i < m) acc[i] += __shfl_xor_sync(0xffffffffu, acc[i + m], o);
+        if (i < m) acc[i] += __shfl_xor_sync(0xffffffffu, acc[i + m], o * GROUPS);
     }
     {
       float* dst = meet + (part * RUN + slice) * L::token + cl;
@@ -473,7 +478,7 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
       }
       u += u2;
       o += o2;
-      us[t * COLS + c] = pack2f(u, u);
+      us[t * COLS + c] = u;
       if (base + t < t1 && col0 + c < p.vdim) p.out[(size_t)(base + t) * p.ldo + (size_t)head * p.vdim + col0 + c] = o;
     }
     asm volatile("cp.async.wait_group 1;\n");
@@ -484,15 +489,16 @@ __global__ void __launch_bounds__(32 * PARTS) delta_runs_kernel(const DeltaArgs 
     for (int k = 0; k < ROWS / 2; ++k)
 #pragma unroll
       for (int c = 0; c < NC; ++c) S[k][c] = mul2(g2, S[k][c]);
-    ulonglong2 u[RUN];  // both columns' (u, u) of token t ^ slice
+    float2 u[RUN];  // both columns of token t ^ slice
 #pragma unroll
-    for (int t = 0; t < RUN; ++t) u[t] = *reinterpret_cast<const ulonglong2*>(us + (t ^ slice) * COLS + cl);
+    for (int t = 0; t < RUN; ++t) u[t] = *reinterpret_cast<const float2*>(us + (t ^ slice) * COLS + cl);
 #pragma unroll
     for (int t = 0; t < RUN; ++t) {
-      S[0][0] = fma2(kr[t].x, u[t].x, S[0][0]);
-      S[0][1] = fma2(kr[t].x, u[t].y, S[0][1]);
-      S[1][0] = fma2(kr[t].y, u[t].x, S[1][0]);
-      S[1][1] = fma2(kr[t].y, u[t].y, S[1][1]);
+      const f32x2 ua = pack2f(u[t].x, u[t].x), ub = pack2f(u[t].y, u[t].y);
+      S[0][0] = fma2(kr[t].x, ua, S[0][0]);
+      S[0][1] = fma2(kr[t].x, ub, S[0][1]);
+      S[1][0] = fma2(kr[t].y, ua, S[1][0]);
+      S[1][1] = fma2(kr[t].y, ub, S[1][1]);
     }
   }
   asm volatile("cp.async.wait_group 0;\n");
